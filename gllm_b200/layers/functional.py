@@ -27,10 +27,11 @@ def linear(x, w, bias=None, out=None):
     return ref.linear(x, w, bias)
 
 
-def linear_silu_mul(x, w_interleaved):
+def linear_silu_mul(x, w_interleaved, out=None):
     if x.is_cuda:
-        return _sm().linear_silu_mul(x, w_interleaved)
-    return ref.linear_silu_mul(x, w_interleaved)
+        return _sm().linear_silu_mul(x, w_interleaved, out)
+    y = ref.linear_silu_mul(x, w_interleaved)
+    return y if out is None else out.copy_(y)
 
 
 def rmsnorm(x, w, eps, residual=None, out=None):
@@ -127,9 +128,9 @@ def embedding_scaled(ids, table, scale):
 
 
 def resid_norm(x, y, w_post, add, w_pre, eps, out_dtype, emit_plain=False, post_scale=None, w_offset=0.0,
-               out_mul=1.0):
+               out_mul=1.0, y_mul=1.0):
     fn = _seq().resid_norm if x.is_cuda else ref.resid_norm
-    return fn(x, y, w_post, add, w_pre, eps, out_dtype, emit_plain, post_scale, w_offset, out_mul)
+    return fn(x, y, w_post, add, w_pre, eps, out_dtype, emit_plain, post_scale, w_offset, out_mul, y_mul)
 
 
 def qk_norm_kv_write(qk, num_heads, num_kv_heads, dim, q_norm_w, k_norm_w, eps, k_cache, v_cache, slots):
@@ -179,27 +180,37 @@ def postnorm(x, y, alpha, w, eps, out_dtype):
 
 
 def qk_norm_rope_kv_write(qkv, num_heads, num_kv_heads, dim, v_dim, q_norm_w, k_norm_w, eps, positions, rot_dims,
-                          rot_base, k_cache, v_cache, slots, freqs=None, mag=1.0):
+                          rot_base, k_cache, v_cache, slots, freqs=None, mag=1.0, unit_norm=False, angles=None,
+                          v_angles=None):
     """num_kv_heads == 0: the rows hold queries only (keys and values are another layer's); `freqs` (fp64 per
-    pair) and `mag`: scaled rotary frequencies and the factor on cos / sin."""
+    pair) and `mag`: scaled rotary frequencies and the factor on cos / sin. `unit_norm`: q / k divided by their root
+    mean square per head, no weight. `angles` (`rotary_angles`): the rows' cos / sin, formed once per step instead of
+    in every layer; `v_angles`: rotate the values over their whole width as well."""
     fn = _seq().qk_norm_rope_kv_write if qkv.is_cuda else ref.qk_norm_rope_kv_write
     return fn(qkv, num_heads, num_kv_heads, dim, v_dim, q_norm_w, k_norm_w, eps, positions, rot_dims, rot_base,
-              k_cache, v_cache, slots, freqs, mag)
+              k_cache, v_cache, slots, freqs, mag, unit_norm, angles, v_angles)
+
+
+def rotary_angles(positions, freqs):
+    """[T, 2 n] fp32 (cos | sin) of position * freqs[i]; freqs fp64 [n]."""
+    return _ssd().rotary_angles(positions, freqs) if positions.is_cuda else ref.rotary_angles(positions, freqs)
 
 
 def masked_attention(q, k_cache, v_cache, inp, scale, num_q_heads, head_dim, v_dim, window=None, chunk=None, sink=None,
-                     out_scale=1.0, out=None, softcap=0.0):
+                     out_scale=1.0, out=None, softcap=0.0, dist_bias=None, gate=None, v_turn=None):
     """Paged causal attention with a sliding window and / or a chunk mask, values of their own width, an optional
-    per-head sink logit in the denominator and an optional tanh cap on the scaled scores."""
+    per-head sink logit in the denominator and an optional tanh cap on the scaled scores. `dist_bias` (r1, r2):
+    r1[h] ln(1 + r2[h] (i - j)) off the scores; `v_turn`: the results of rotated values turned back by the query's
+    angle; `gate`: results times sigmoid(gate)."""
     if q.is_cuda:
         return _seq().window_attention(q, k_cache, v_cache, inp.block_table, inp.seq_lens, inp.query_start_loc,
                                        inp.positions, scale, num_q_heads, head_dim, window, sink,
                                        num_decode_seqs=inp.padded_tokens or inp.num_decode_seqs,
                                        max_q_len=inp.max_q_len, chunk=chunk, v_dim=v_dim, out_scale=out_scale, out=out,
-                                       softcap=softcap)
+                                       softcap=softcap, dist_bias=dist_bias, gate=gate, v_turn=v_turn)
     return ref.window_attention(q, k_cache, v_cache, inp.block_table, inp.seq_lens, inp.query_start_loc, scale,
                                 num_q_heads, head_dim, window, sink, chunk=chunk, v_dim=v_dim, out_scale=out_scale,
-                                out=out, softcap=softcap)
+                                out=out, softcap=softcap, dist_bias=dist_bias, gate=gate, v_turn=v_turn)
 
 
 def linear_state_scan(q, k, v, beta, a, neg_a, dt_bias, decay, state, inp, heads, qk_heads, dim, v_dim, silu_in,
@@ -215,12 +226,12 @@ def gated_group_norm(o, gate, w, group, eps, act, out_scale=1.0, out=None, out_d
     return fn(o, gate, w, group, eps, act, out_scale, out, out_dtype)
 
 
-def silu_mul(gu):
+def silu_mul(gu, out=None):
     if gu.is_cuda:
-        if gu.dtype == torch.bfloat16 and gu.is_contiguous():
+        if gu.dtype == torch.bfloat16 and gu.is_contiguous() and out is None:
             return _sm().silu_and_mul(gu)
-        return _seq().silu_mul(gu)
-    return ref.silu_mul(gu)
+        return _seq().silu_mul(gu, out)
+    return ref.silu_mul(gu) if out is None else out.copy_(ref.silu_mul(gu))
 
 
 def router_topk(h, w, top_k):
@@ -333,3 +344,32 @@ def routed_relu2_experts(h, w1, w2, weights, ids, grouped):
     if h.is_cuda:
         return _pair().routed_relu2_experts(h, w1, w2, weights, ids, grouped)
     return ref.routed_relu2_experts(h, w1, w2, weights, ids)
+
+
+# -- Mamba-2 recurrence, gate before a grouped norm, per-layer token input (csrc/seq/ssd_ops.cu) ----------------
+def _ssd():
+    from gllm_b200.ops import sm100_ssd
+    return sm100_ssd
+
+
+def ssd_scan(x, b, c, dt, neg_a, dt_bias, d_skip, state, inp, heads, groups, nstate, v_dim):
+    """y [T, heads * v_dim] fp32 of the Mamba-2 recurrence; x, b, c, dt are column slices of wider rows."""
+    slots = inp.rec_slots if state is not None else None
+    if x.is_cuda:
+        return _ssd().ssd_scan(x, b, c, dt, neg_a, dt_bias, d_skip, state, slots, inp.seq_lens, inp.query_start_loc,
+                               heads, groups, nstate, v_dim,
+                               num_decode_seqs=inp.padded_tokens or inp.num_decode_seqs, max_q_len=inp.max_q_len)
+    return ref.ssd_scan(x, b, c, dt, neg_a, dt_bias, d_skip, state, slots, inp.seq_lens, inp.query_start_loc, heads,
+                        groups, nstate, v_dim)
+
+
+def gate_then_norm(o, gate, w, group, eps, out=None, out_dtype=None):
+    """RMS norm over groups of columns of o * silu(gate), times w."""
+    fn = _ssd().gate_then_norm if o.is_cuda else ref.gate_then_norm
+    return fn(o, gate, w, group, eps, out, out_dtype)
+
+
+def gelu_gate_embed(g, ids, table, col0):
+    """gelu_tanh(g) times the columns [col0, col0 + dim) of the tokens' table rows."""
+    fn = _ssd().gelu_gate_embed if g.is_cuda else ref.gelu_gate_embed
+    return fn(g, ids, table, col0)

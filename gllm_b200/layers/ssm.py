@@ -7,6 +7,11 @@ y = gelu_tanh(W_y h + b_y) and u = causal depthwise convolution of (W_x h + b_x)
 width / blocks channels two gates r = sigmoid(A_r u + b_r), i = sigmoid(A_i u + b_i) (block-diagonal maps);
 a = exp(-c r softplus(lam)), S <- a S + sqrt(1 - a^2) i u from S = 0; output projection of S * y.
 
+`Mamba2Core` (a core in the sense of layers/parallel_mixer.py): one projection gives [z | x | B | C | dt]; x, B and C
+pass one causal depthwise convolution with bias + SiLU; per head dt = softplus(dt + dt_bias),
+S <- exp(-exp(A_log) dt) S + dt B x^T with S [state, v_dim] and B, C shared by the heads of a group,
+y = S^T C + D x; then y * SiLU(z), RMS norm in `norm_groups` equal parts, weight.
+
 Per-sequence state lives in slot-indexed device tensors owned by the engine's cache (one set per layer run):
 the last taps - 1 convolution inputs and the fp32 [state, channels] recurrence matrix. A chunk that starts at
 position 0 starts from zeros, any other chunk continues from its slot.
@@ -104,3 +109,52 @@ class RGLRUMixer(nn.Module):
                                     reader.get(pre + "ri.b").float().reshape(nb, bw)], 1).reshape(-1))
         put(self.c_decay, -self.decay_scale * torch.nn.functional.softplus(reader.get(pre + "lam").float()))
         put(self.o_w, reader.get(pre + "o"))
+
+
+class Mamba2Core(nn.Module):
+    uses_pages, uses_state = False, True
+    in_names = ("in",)
+
+    def __init__(self, heads: int, groups: int, nstate: int, v_dim: int, taps: int, norm_groups: int, eps: float, dtype,
+                 device):
+        super().__init__()
+        assert heads % groups == 0 and (heads * v_dim) % norm_groups == 0, (heads, groups, v_dim, norm_groups)
+        self.heads, self.groups, self.nstate, self.v_dim, self.taps, self.eps = heads, groups, nstate, v_dim, taps, eps
+        self.inner, self.n_bc = heads * v_dim, groups * nstate
+        self.n_conv = self.inner + 2 * self.n_bc
+        self.norm_part = self.inner // norm_groups
+        self.in_rows = (self.inner + self.n_conv + heads,)
+        self.n_in, self.n_out = self.in_rows[0], self.inner
+
+        def par(*shape, dt=torch.float32):
+            return nn.Parameter(torch.zeros(*shape, dtype=dt, device=device), requires_grad=False)
+
+        self.conv_w = par(self.n_conv, taps)
+        self.conv_b = par(self.n_conv)
+        self.neg_a = par(heads)                      # -exp(A_log)
+        self.dt_bias = par(heads)
+        self.d_skip = par(heads)
+        self.norm_w = par(self.inner)
+
+    def cache_entry(self):
+        return {"kind": "linear", "heads": self.heads, "dim": self.nstate, "vdim": self.v_dim, "taps": self.taps,
+                "channels": self.n_conv}
+
+    def core(self, inp, proj, cache, run_id, out, out_scale=1.0):
+        assert out_scale == 1.0, "a norm precedes the output: fold the scale into its weight"
+        conv_state = cache.conv_state[run_id] if cache is not None else None
+        state = cache.ssm_state[run_id] if cache is not None else None
+        ni, nb, nc = self.inner, self.n_bc, self.n_conv
+        xbc = Fn.causal_conv_silu(proj[:, ni:], nc, self.conv_w, self.conv_b, conv_state, inp)
+        y = Fn.ssd_scan(xbc[:, :ni], xbc[:, ni:ni + nb], xbc[:, ni + nb:nc], proj[:, ni + nc:ni + nc + self.heads],
+                        self.neg_a, self.dt_bias, self.d_skip, state, inp, self.heads, self.groups, self.nstate,
+                        self.v_dim)
+        return Fn.gate_then_norm(y, proj[:, :ni], self.norm_w, self.norm_part, self.eps, out)
+
+    def load_extra(self, reader, pre, put):
+        put(self.conv_w, reader.get(pre + "conv").float())
+        put(self.conv_b, reader.get(pre + "conv.b").float())
+        put(self.neg_a, -torch.exp(reader.get(pre + "A_log").float()))
+        put(self.dt_bias, reader.get(pre + "dt_bias").float())
+        put(self.d_skip, reader.get(pre + "D").float())
+        put(self.norm_w, reader.get(pre + "norm").float())

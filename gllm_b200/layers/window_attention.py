@@ -68,14 +68,24 @@ class RotaryChunkCore(nn.Module):
       * values of their own width `v_dim`;
       * `bias`: the q / k / v projections have biases (the mixer adds them in the joint projection);
       * `kv_from` (a layer index): the core has no key / value projections and no cache of its own; it reads the
-        pages that layer wrote (rotated keys, values) with its own queries and mask.
+        pages that layer wrote (rotated keys, values) with its own queries and mask;
+      * `unit_qk`: q and k are divided by their root mean square per head, without a weight (a rotation keeps that
+        norm, so the order of the two does not matter);
+      * `turn_values`: the value of position j is rotated by j over its whole width (entry m with m + v_dim / 2,
+        frequencies of `rot_base` over v_dim, unscaled) and cached so; the result at position i is turned back by i;
+      * `dist_bias`: r1[h] ln(1 + r2[h] (i - j)) is taken off the scaled score (per-head numbers 'r1', 'r2');
+      * `out_gate`: the heads' results are multiplied by sigmoid of one more projection of the input ('g');
+      * `rot_scaling` with {factor, low, high, original}: the frequency bands of `ops.ref.banded_rotary_frequencies`.
+    With `unit_qk` or `turn_values` the cos / sin rows come from `inp.angles` (formed once per step by the model, see
+    `angle_tables`) instead of from every layer's own kernel.
     A core in the sense of layers/parallel_mixer.py: it reads [q | k | v] rows of a joint projection."""
     uses_pages, uses_state = True, False
 
     def __init__(self, heads: int, kv_heads: int, dim: int, v_dim: int, scale: float, rot_dims: int, rot_base: float,
                  chunk: Optional[int], window: Optional[int], eps: float, dtype, device, qk_norm: bool = True,
                  rot_scaling: Optional[dict] = None, softcap: float = 0.0, unit_sink: bool = False,
-                 bias: bool = False, kv_from: Optional[int] = None):
+                 bias: bool = False, kv_from: Optional[int] = None, unit_qk: bool = False, turn_values: bool = False,
+                 dist_bias: bool = False, out_gate: bool = False):
         super().__init__()
         assert heads % kv_heads == 0, (heads, kv_heads)
         assert rot_dims % 2 == 0 and rot_dims <= dim, (rot_dims, dim)
@@ -89,14 +99,31 @@ class RotaryChunkCore(nn.Module):
         else:
             self.in_names = ("q",)
             self.in_rows = (heads * dim,)
+        self.unit_qk, self.turn_values, self.out_gate = bool(unit_qk), bool(turn_values), bool(out_gate)
+        assert not (unit_qk and qk_norm) and not ((unit_qk or turn_values) and kv_from is not None)
+        assert not turn_values or v_dim % 2 == 0, v_dim
+        if out_gate:
+            self.in_names += ("g",)
+            self.in_rows += (heads * v_dim,)
+        if dist_bias:
+            self.r1 = nn.Parameter(torch.zeros(heads, dtype=torch.float32, device=device), requires_grad=False)
+            self.r2 = nn.Parameter(torch.zeros(heads, dtype=torch.float32, device=device), requires_grad=False)
+        else:
+            self.r1 = self.r2 = None
         self.n_in, self.n_out = sum(self.in_rows), heads * v_dim
         self.q_norm_w = nn.Parameter(torch.zeros(dim, dtype=dtype, device=device), requires_grad=False) if qk_norm \
             else None
         self.k_norm_w = nn.Parameter(torch.zeros(dim, dtype=dtype, device=device), requires_grad=False) if qk_norm \
             else None
         self.mag = 1.0
-        if rot_scaling and rot_dims > 0:
-            from gllm_b200.ops import ref
+        from gllm_b200.ops import ref
+        self.step_angles = self.unit_qk or self.turn_values or bool(rot_scaling and "low" in rot_scaling)
+        if self.step_angles:
+            self.register_buffer("freqs", ref.banded_rotary_frequencies(rot_dims, rot_base, rot_scaling).to(device),
+                                 persistent=False)
+            self.register_buffer("v_freqs", ref.banded_rotary_frequencies(v_dim, rot_base).to(device)
+                                 if turn_values else None, persistent=False)
+        elif rot_scaling and rot_dims > 0:
             f, self.mag = ref.pair_rotary_frequencies(rot_dims, rot_base, rot_scaling, dtype=torch.float64)
             self.register_buffer("freqs", f.to(device), persistent=False)
         else:
@@ -111,12 +138,46 @@ class RotaryChunkCore(nn.Module):
             return {"kind": "shared", "layer": int(self.kv_from)}
         return {"kind": "kv", "heads": self.kv_heads, "dim": self.dim, "vdim": self.v_dim}
 
+    def angle_tables(self):
+        """[(key, fp64 frequencies)] of the cos / sin rows this core reads from `inp.angles`; equal keys are equal
+        tables, so layers that rotate alike share one."""
+        if not self.step_angles:
+            return []
+        out = [(self._angle_key(f), f) for f in (self.freqs, self.v_freqs) if f is not None and f.numel()]
+        return out
+
+    @staticmethod
+    def _angle_key(f):
+        return tuple(f.tolist())
+
+    def _angles(self, inp, name):
+        f = getattr(self, name)
+        if f is None or not f.numel():
+            return None
+        if name not in self.__dict__.setdefault("_keys", {}):
+            self._keys[name] = self._angle_key(f)
+        tabs = getattr(inp, "angles", None)
+        if tabs is not None and self._keys[name] in tabs:
+            return tabs[self._keys[name]]
+        return Fn.rotary_angles(inp.positions, f)          # a core driven without its model
+
     def core(self, inp, proj, cache, run_id, out, out_scale=1.0):
         if cache is None:      # memory probe without a cache
             out.zero_()
             return out
         kc, vc = cache.k_cache[run_id], cache.v_cache[run_id]
         own = self.kv_from is None
+        if self.step_angles or self.r1 is not None or self.out_gate:
+            ang = self._angles(inp, "freqs") if self.step_angles else None
+            v_ang = self._angles(inp, "v_freqs") if self.step_angles else None
+            q = Fn.qk_norm_rope_kv_write(proj, self.heads, self.kv_heads if own else 0, self.dim, self.v_dim,
+                                         self.q_norm_w, self.k_norm_w, self.eps, inp.positions, self.rot_dims,
+                                         self.rot_base, kc, vc, inp.slot_mapping, None if self.step_angles
+                                         else self.freqs, self.mag, self.unit_qk, ang, v_ang)
+            gate = proj[:, self.n_in - self.n_out:self.n_in] if self.out_gate else None
+            return Fn.masked_attention(q, kc, vc, inp, self.scale, self.heads, self.dim, self.v_dim, self.window,
+                                       self.chunk, self.sink, out_scale, out, self.softcap,
+                                       (self.r1, self.r2) if self.r1 is not None else None, gate, v_ang)
         q = Fn.qk_norm_rope_kv_write(proj, self.heads, self.kv_heads if own else 0, self.dim, self.v_dim,
                                      self.q_norm_w, self.k_norm_w, self.eps, inp.positions, self.rot_dims,
                                      self.rot_base, kc, vc, inp.slot_mapping, self.freqs, self.mag)
@@ -127,3 +188,6 @@ class RotaryChunkCore(nn.Module):
         if self.q_norm_w is not None:
             put(self.q_norm_w, reader.get(pre + "q.norm"))
             put(self.k_norm_w, reader.get(pre + "k.norm"))
+        if getattr(self, "r1", None) is not None:
+            put(self.r1, reader.get(pre + "r1").float())
+            put(self.r2, reader.get(pre + "r2").float())

@@ -9,7 +9,12 @@ with identity experts and a shared expert); and sandwich blocks whose norm weigh
 `Notadra`: rotary attention with biased projections, YaRN-scaled partial rotation, capped scores, a unit sink in the
 softmax denominator, values of their own width and layers that read an earlier layer's keys and values; a
 sigmoid-scored, group-limited mixture of ungated squared-ReLU experts; a hashed embedding of the (previous, current)
-token pair added to the token embedding; logits scaled through the final norm):
+token pair added to the token embedding; logits scaled through the final norm); and parallel blocks (architecture
+`Vikupel`: Mamba-2 mixers, windowed attention with a logarithmic distance bias and an output gate, rotary attention with
+rotated values, gated SiLU feed-forward beside the mixer, a residual multiplier, a gated per-layer token embedding after
+every layer, a loop whose passes share weights).
+
+The branch-norm form:
 
     x = embed[token]
     per layer:  x += ls1 * rms(mixer(x)) * n1 ;  x += ls2 * rms(ff(x)) * n2            (sublayers read x itself)
@@ -45,12 +50,24 @@ Notadra (the sandwich form with gains 1 + w):
     per layer:  x += rms(mixer(rms(x) (1 + n1))) (1 + n1b) ;  x += rms(ff(rms(x) (1 + n2))) (1 + n2b)
     logits = head @ (logit_scale * rms(x) (1 + final_norm))
 
-config.json keys read here: architecture, vocab, width, embedding.scale, embedding.bigram.{buckets, mul_prev,
+The parallel form (mult: the residual multiplier; one norm feeds both sublayers; the side line only with a token side):
+
+    x = embed[token]
+    per layer:  h = rms(x) * n1 ;  x += mult * (mixer(h) + ff(h))
+                x += mult * rms(P (gelu_tanh(G x) * side[token, layer])) * ns
+    loop: the span's passes follow each other, each with its own cache entries; nothing happens in between
+    logits = head @ (rms(x) * final_norm)
+
+Here mixer and feed-forward share one output GEMM (`CoreMixer` with a `GatedBranch`), so the stream update is
+x += mult * y in one kernel that also emits x in the compute dtype for G; the second update (norm of the side branch,
+multiplier, next layer's norm1) is one kernel as in the sandwich form.
+
+config.json keys read here: architecture, vocab, width, residual_mult, token_side.dim, embedding.scale, embedding.bigram.{buckets, mul_prev,
 mul_cur}, logit_scale, layers[i].mixer.{kv_from, softcap, rot.scaling.{factor, original, fast, slow}},
 norm.eps, loop.{start,stop,times},
 postln_alpha, logit_softcap, layers[i].{type, mixer{...}, mlp{kind, ff | expert.{ff, limit}, router.{experts, top,
 identity, scale, groups.{count, keep}}, shared.{ff, limit}} | null}, optional torch_dtype. Tensor names: embed, bigram,
-head, l<i>.mix.{q,k,v}.b, l<i>.mlp.e<j>.{up,down}, final.norm, l<i>.norm1|norm1b|norm2|norm2b|ls1|ls2, l<i>.mix.*, l<i>.mlp.up|down|gate|router|correction|
+head, side.embed, l<i>.side.{gate,proj,norm}, l<i>.mix.{q,k,v}.b, l<i>.mlp.e<j>.{up,down}, final.norm, l<i>.norm1|norm1b|norm2|norm2b|ls1|ls2, l<i>.mix.*, l<i>.mlp.up|down|gate|router|correction|
 e<j>.{gate,up,down}|shared.{gate,up,down}.
 """
 from __future__ import annotations
@@ -66,7 +83,7 @@ from gllm_b200.layers.latent_attention import LatentAttention
 from gllm_b200.layers.linear_attention import DecayLinearCore, GatedDeltaCore, KeyDecayLinearCore
 from gllm_b200.layers.moe import GroupedGLUMoE, GroupedRelu2MoE, SelectedSoftmaxMoE
 from gllm_b200.layers.parallel_mixer import CoreMixer
-from gllm_b200.layers.ssm import Mamba1Mixer, RGLRUMixer
+from gllm_b200.layers.ssm import Mamba1Mixer, Mamba2Core, RGLRUMixer
 from gllm_b200.layers.window_attention import RotaryChunkCore, SinkWindowAttention
 from gllm_b200.parallel import state as ps
 
@@ -86,7 +103,8 @@ class HybridSpec:
     loop_stop: int = 0
     loop_times: int = 1
     dtype: torch.dtype = torch.bfloat16
-    # "sandwich": x += post(f(pre(x))) | "postnorm": x <- norm(alpha x + f(x)) | "branchnorm": x += ls * post(f(x))
+    # "sandwich": x += post(f(pre(x))) | "postnorm": x <- norm(alpha x + f(x)) | "branchnorm": x += ls * post(f(x)) |
+    # "parallel": x += mult (mixer(pre(x)) + ff(pre(x)))
     block: str = "sandwich"
     resid_alpha: float = 1.0
     logit_softcap: float = 0.0         # 0: none
@@ -97,6 +115,9 @@ class HybridSpec:
     logit_scale: float = 1.0
     # {"buckets", "mul_prev", "mul_cur"}: a second embedding table indexed by a hash of the (previous, current) pair
     pair_hash: Optional[dict] = None
+    resid_mult: float = 1.0            # parallel blocks: factor on everything that is added to the stream
+    loop_readd: bool = True            # the embedding output is added before every pass of the loop but the first
+    token_side_dim: int = 0            # width of the per-layer token input (0: none)
     eos_token_id: Optional[object] = None
     use_mla: bool = False
     quant: Optional[str] = None
@@ -152,13 +173,27 @@ def spec_notadra(cfg) -> HybridSpec:
                       eos_token_id=cfg.get("eos_token_id"))
 
 
-def layer_runs(n_layers: int, start: int, stop: int, times: int):
-    """[(layer index, add_embed)] in execution order; add_embed marks the first layer of every pass but the first."""
+def spec_vikupel(cfg) -> HybridSpec:
+    loop, side = cfg.get("loop") or {}, cfg.get("token_side") or {}
+    dt = cfg.get("torch_dtype", cfg.get("dtype", "bfloat16"))
+    if dt not in _DTYPES:
+        raise ValueError(f"unsupported dtype {dt} for this architecture (bfloat16 | float32)")
+    return HybridSpec(arch="vikupel", hidden_size=int(cfg["width"]), vocab_size=int(cfg["vocab"]),
+                      rms_eps=float(cfg["norm"]["eps"]), embed_scale=1.0, layers=[dict(x) for x in cfg["layers"]],
+                      loop_start=int(loop.get("start", 0)), loop_stop=int(loop.get("stop", 0)),
+                      loop_times=int(loop.get("times", 1)), loop_readd=False, dtype=_DTYPES[dt], block="parallel",
+                      ff_act="silu_gate", resid_mult=float(cfg.get("residual_mult", 1.0)),
+                      token_side_dim=int(side.get("dim", 0)), eos_token_id=cfg.get("eos_token_id"))
+
+
+def layer_runs(n_layers: int, start: int, stop: int, times: int, readd: bool = True):
+    """[(layer index, add_embed)] in execution order; add_embed marks the first layer of every pass but the first
+    (never without `readd`)."""
     if times <= 1 or stop <= start:
         return [(i, False) for i in range(n_layers)]
     runs = [(i, False) for i in range(start)]
     for r in range(times):
-        runs += [(i, r > 0 and i == start) for i in range(start, stop)]
+        runs += [(i, readd and r > 0 and i == start) for i in range(start, stop)]
     return runs + [(i, False) for i in range(stop, n_layers)]
 
 
@@ -174,8 +209,30 @@ class Relu2MLP(nn.Module):
         return Fn.linear_any(Fn.relu2(Fn.linear_any(h, self.up_w)), self.down_w)
 
 
+def make_parallel_mixer(kind: str, m: dict, ff: int, spec: HybridSpec, device):
+    """Mixer of a parallel block with the feed-forward (width ff, 0 = none) as one more branch."""
+    h, dt, eps = spec.hidden_size, spec.dtype, spec.rms_eps
+    if kind == "mamba2":
+        core = Mamba2Core(int(m["heads"]), int(m.get("groups", 1)), int(m["state"]), int(m["vdim"]),
+                          int(m.get("conv", 1)), int(m.get("norm_groups", 1)), eps, dt, device)
+    elif kind in ("attention", "attention_2"):
+        rot, window = m.get("rot") or {}, (m.get("mask") or {}).get("size")
+        plain = kind == "attention"                    # no rotation; distance bias and output gate
+        core = RotaryChunkCore(int(m["heads"]), int(m.get("kv_heads", m["heads"])), int(m["dim"]),
+                               int(m.get("vdim", m["dim"])), float(m["scale"]),
+                               0 if plain else int(rot.get("dims", m["dim"])), float(rot.get("base", 10000.0)), None,
+                               int(window) if plain and window is not None else None, eps, dt, device, qk_norm=False,
+                               rot_scaling=None if plain else rot.get("scaling"), unit_qk=not plain,
+                               turn_values=not plain, dist_bias=plain, out_gate=plain)
+    else:
+        raise ValueError(f"unknown mixer type {kind!r}")
+    return CoreMixer(h, [core], [""], [1.0], dt, device, ff=ff)
+
+
 def make_mixer(kind: str, m: dict, spec: HybridSpec, device):
     h, dt = spec.hidden_size, spec.dtype
+    if spec.block == "parallel":
+        return make_parallel_mixer(kind, m, 0, spec, device)
     if kind == "attention" and spec.arch == "notadra":
         rot = m.get("rot") or {}
         src = m.get("kv_from")
@@ -291,6 +348,18 @@ class HybridLayer(nn.Module):
 
         self.norm1_w, self.norm1b_w = norm(), (norm() if sandwich else None)
         self.ls1 = scale() if scaled else None
+        self.side_gate_w = self.side_proj_w = self.side_norm_w = None
+        if spec.block == "parallel":
+            mlp = L.get("mlp")
+            assert mlp is None or mlp.get("kind", "dense") == "dense", mlp
+            self.mixer = make_parallel_mixer(L["type"], L["mixer"], int(mlp["ff"]) if mlp else 0, spec, device)
+            self.mlp = None                            # a branch of the mixer's joint output product
+            if spec.token_side_dim:
+                d = spec.token_side_dim
+                self.side_gate_w = nn.Parameter(torch.zeros(d, h, dtype=dt, device=device), requires_grad=False)
+                self.side_proj_w = nn.Parameter(torch.zeros(h, d, dtype=dt, device=device), requires_grad=False)
+                self.side_norm_w = norm()
+            return
         self.mixer = make_mixer(L["type"], L["mixer"], spec, device)
         mlp = L.get("mlp")
         if mlp is not None:
@@ -316,10 +385,17 @@ class HybridLM(nn.Module):
         self.embed_w = nn.Parameter(torch.zeros(spec.vocab_size, h, dtype=dt, device=device), requires_grad=False)
         self.pair_w = nn.Parameter(torch.zeros(spec.pair_hash["buckets"] + 1, h, dtype=dt, device=device),
                                    requires_grad=False) if spec.pair_hash else None
+        self.side_w = nn.Parameter(torch.zeros(spec.vocab_size, spec.num_layers * spec.token_side_dim, dtype=dt,
+                                               device=device), requires_grad=False) if spec.token_side_dim else None
         self.layers = nn.ModuleList([HybridLayer(spec, i, device) for i in range(spec.num_layers)])
         self.final_norm_w = nn.Parameter(torch.ones(h, dtype=dt, device=device), requires_grad=False)
         self.lm_head_w = nn.Parameter(torch.zeros(spec.vocab_size, h, dtype=dt, device=device), requires_grad=False)
-        self.runs = layer_runs(spec.num_layers, spec.loop_start, spec.loop_stop, spec.loop_times)
+        self.runs = layer_runs(spec.num_layers, spec.loop_start, spec.loop_stop, spec.loop_times, spec.loop_readd)
+        # cos / sin rows that layers read instead of forming them: one table per distinct set of frequencies and step
+        self.angle_tables = {}
+        for l in self.layers:
+            for c in getattr(l.mixer, "cores", []):
+                self.angle_tables.update(dict(c.angle_tables()) if hasattr(c, "angle_tables") else {})
         # the pair embedding keeps every sequence's last token in its state slot
         self.has_state = any(getattr(l.mixer, "uses_state", not l.mixer.uses_pages) for l in self.layers) or \
             spec.pair_hash is not None
@@ -362,6 +438,8 @@ class HybridLM(nn.Module):
             return self._forward_postnorm(inp, cache), None
         if spec.block == "branchnorm":
             return self._forward_branchnorm(inp, cache), None
+        if spec.block == "parallel":
+            return self._forward_parallel(inp, cache), None
         off = spec.norm_offset
         if spec.pair_hash is not None:
             ph = spec.pair_hash
@@ -433,6 +511,31 @@ class HybridLM(nn.Module):
             h = Fn.resid_norm(x, None, None, None, self.final_norm_w, eps, dt)
         return h
 
+    def _forward_parallel(self, inp, cache):
+        """One norm feeds mixer and feed-forward, whose sum arrives as one product; x += mult * y, then the per-layer
+        token input reads the new stream and adds mult * rms(side) * ns."""
+        spec, eps, dt, mult = self.spec, self.spec.rms_eps, self.spec.dtype, self.spec.resid_mult
+        inp.angles = {k: Fn.rotary_angles(inp.positions, f) for k, f in self.angle_tables.items()}
+        x = Fn.embedding_scaled(inp.tokens, self.embed_w, 1.0)
+        n, d = len(self.runs), spec.token_side_dim
+        h = Fn.resid_norm(x, None, None, None, self.layers[self.runs[0][0]].norm1_w if n else self.final_norm_w, eps, dt)
+        for r, (li, _) in enumerate(self.runs):
+            L = self.layers[li]
+            y, w_post = L.mixer(inp, h, cache, r), None
+            w_next = self.final_norm_w if r + 1 == n else self.layers[self.runs[r + 1][0]].norm1_w
+            if d:
+                xs = Fn.resid_norm(x, y, None, None, None, eps, dt, emit_plain=True, y_mul=mult)
+                g = Fn.gelu_gate_embed(Fn.linear_any(xs, L.side_gate_w), inp.tokens, self.side_w, li * d)
+                y, w_post = Fn.linear_any(g, L.side_proj_w), L.side_norm_w
+            if self.trace is not None:
+                Fn.resid_norm(x, y, w_post, None, None, eps, dt, y_mul=mult)
+                self.trace.append(x.clone())
+                h = Fn.resid_norm(x, None, None, None, w_next, eps, dt)
+            else:
+                h = Fn.resid_norm(x, y, w_post, None, w_next, eps, dt, y_mul=mult)
+        inp.angles = None
+        return h
+
     def compute_logits(self, inp, hidden, tpc=None, all_rows: bool = False, local: bool = False):
         rows = hidden if all_rows else hidden.index_select(0, inp.logits_idx.long())
         z = Fn.linear_any(rows, self.lm_head_w)
@@ -464,6 +567,12 @@ class HybridLM(nn.Module):
                 p.data.copy_(-torch.exp(torch.rand(p.shape, generator=g) * 2.0 - 1.0))
             elif name.endswith("dt_b"):
                 p.data.copy_(torch.rand(p.shape, generator=g) * 2.0 - 3.0)
+            elif name.endswith(".r1"):
+                p.data.copy_(torch.rand(p.shape, generator=g) + 0.5)
+            elif name.endswith(".r2"):
+                p.data.copy_(torch.rand(p.shape, generator=g) * 0.2 + 0.01)
+            elif "cores" in name and name.endswith("norm_w") or name.endswith("side_norm_w"):
+                p.data.fill_(1.0)
             elif name.endswith("d_skip"):
                 p.data.fill_(1.0)
             elif name.endswith("neg_a"):
@@ -491,6 +600,8 @@ class HybridLM(nn.Module):
         put(self.embed_w, reader.get("embed"))
         if self.pair_w is not None:
             put(self.pair_w, reader.get("bigram"))
+        if self.side_w is not None:
+            put(self.side_w, reader.get("side.embed"))
         for n, L in enumerate(self.layers):
             pre = f"l{L.layer_id}."
             put(L.norm1_w, reader.get(pre + "norm1"))
@@ -498,6 +609,10 @@ class HybridLM(nn.Module):
                 put(L.norm1b_w, reader.get(pre + "norm1b"))
             m = L.mixer
             mp = pre + "mix."
+            if L.side_gate_w is not None:
+                put(L.side_gate_w, reader.get(pre + "side.gate"))
+                put(L.side_proj_w, reader.get(pre + "side.proj"))
+                put(L.side_norm_w, reader.get(pre + "side.norm"))
             if isinstance(m, SinkWindowAttention):
                 put(m.qk_w, torch.cat([reader.get(mp + "q"), reader.get(mp + "k")], 0))
                 if m.q_norm_w is not None:
@@ -517,7 +632,7 @@ class HybridLM(nn.Module):
                 put(m.d_skip, reader.get(mp + "D").float())
                 put(m.o_w, reader.get(mp + "o"))
             elif isinstance(m, CoreMixer):
-                m.load(reader, mp, put)
+                m.load(reader, mp, put, pre + "mlp.")
             elif isinstance(m, (RGLRUMixer, LatentAttention)):
                 m.load(reader, mp, put)
             if L.ls1 is not None:
@@ -576,3 +691,7 @@ def build_bevovik(cfg, device):
 
 def build_notadra(cfg, device):
     return HybridLM(spec_notadra(cfg), device)
+
+
+def build_vikupel(cfg, device):
+    return HybridLM(spec_vikupel(cfg), device)

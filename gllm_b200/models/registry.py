@@ -4,7 +4,7 @@ Supported `architectures[0]` values:
   LlamaForCausalLM, Qwen2ForCausalLM, Qwen3ForCausalLM, Qwen2MoeForCausalLM, Qwen3MoeForCausalLM,
   MixtralForCausalLM, ChatGLMModel / ChatGLMForConditionalGeneration, DeepseekV2ForCausalLM,
   DeepseekV3ForCausalLM, Qwen2_5_VLForConditionalGeneration, Qwen3VLForConditionalGeneration,
-  Qwen3VLMoeForConditionalGeneration, Saritar, Femolix, Bevovik and Notadra (layer-list decoders,
+  Qwen3VLMoeForConditionalGeneration, Saritar, Femolix, Bevovik, Notadra and Vikupel (layer-list decoders,
   models/hybrid.py).
 """
 from __future__ import annotations
@@ -177,6 +177,11 @@ def _build_notadra(cfg, device):
     return build_notadra(cfg, device)
 
 
+def _build_vikupel(cfg, device):
+    from gllm_b200.models.hybrid import build_vikupel
+    return build_vikupel(cfg, device)
+
+
 def _build_femolix(cfg, device):
     from gllm_b200.models.hybrid import build_femolix
     return build_femolix(cfg, device)
@@ -187,6 +192,7 @@ ARCHITECTURES: Dict[str, Callable] = {
     "Femolix": _build_femolix,
     "Bevovik": _build_bevovik,
     "Notadra": _build_notadra,
+    "Vikupel": _build_vikupel,
     "LlamaForCausalLM": _build_decoder(spec_llama),
     "MistralForCausalLM": _build_decoder(spec_llama),
     "Qwen2ForCausalLM": _build_decoder(spec_qwen2),

@@ -467,17 +467,21 @@ def embedding_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float) -> to
 def resid_norm(x: torch.Tensor, y: Optional[torch.Tensor], w_post: Optional[torch.Tensor],
                add: Optional[torch.Tensor], w_pre: Optional[torch.Tensor], eps: float, out_dtype,
                emit_plain: bool = False, post_scale: Optional[torch.Tensor] = None, w_offset: float = 0.0,
-               out_mul: float = 1.0):
+               out_mul: float = 1.0, y_mul: float = 1.0):
     """In place on the fp32 stream x [T, W]:  x += rms(y) * w_post ;  x += add ;  returns rms(x) * w_pre cast to
     `out_dtype` (None when w_pre is None). Every step is optional. All arithmetic in fp32. `post_scale` [W] fp32
     (a layer scale) multiplies the normed branch element by element: x += rms(y) * w_post * post_scale. `emit_plain` (with w_pre None): returns the stream itself rounded to
     `out_dtype` — x for fp32 — for sublayers that read the stream without a norm in front. `w_offset` is added to
     both norm weights in fp32 (1.0 for weights stored around zero); `out_mul` multiplies the normed result before it
-    is rounded (a logit scale folded into the final norm)."""
+    is rounded (a logit scale folded into the final norm). `y_mul` multiplies the branch before it is added (a residual
+    multiplier); without w_post the branch is added as it is, not normed: x += y_mul * y."""
     if y is not None:
-        yf = y.float()
-        br = yf * torch.rsqrt((yf * yf).mean(-1, keepdim=True) + eps) * (w_post.float() + w_offset)
-        x += br * post_scale.float() if post_scale is not None else br
+        br = y.float()
+        if w_post is not None:
+            br = br * torch.rsqrt((br * br).mean(-1, keepdim=True) + eps) * (w_post.float() + w_offset)
+        if post_scale is not None:
+            br = br * post_scale.float()
+        x += br * y_mul
     if add is not None:
         x += add
     if w_pre is None:
@@ -518,13 +522,17 @@ def window_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      seq_lens: torch.Tensor, query_start_loc: torch.Tensor, scale: float, num_q_heads: int,
                      head_dim: int, window: Optional[int], sink: Optional[torch.Tensor],
                      chunk: Optional[int] = None, v_dim: Optional[int] = None, out_scale: float = 1.0,
-                     out: Optional[torch.Tensor] = None, softcap: float = 0.0) -> torch.Tensor:
+                     out: Optional[torch.Tensor] = None, softcap: float = 0.0, dist_bias=None,
+                     gate: Optional[torch.Tensor] = None, v_turn: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal paged attention where position i sees j with 0 <= i - j < window (None: all of the past), and, with
     `chunk`, only j of its own chunk (floor(i / chunk) == floor(j / chunk), counted from position 0); the softmax
     denominator has one more term exp(sink[h]) that carries no value (None: plain softmax). Values may be wider or
     narrower than keys (`v_dim`); the result is multiplied by `out_scale` and written to `out` [T, H * v_dim] (any
     row stride) when given. `softcap` > 0 bounds every scaled score: s <- softcap * tanh(s / softcap), before the
-    mask and the softmax."""
+    mask and the softmax. `dist_bias` = (r1, r2) [H] fp32: r1[h] ln(1 + r2[h] (i - j)) is taken off the score of key j
+    for the query at i. `v_turn` [T, v_dim] fp32 (cos | sin per pair, of the query's position): the values were
+    rotated by their own positions, and every head's result is turned back, pair (m, m + v_dim / 2) by the negative
+    angle. `gate` [T, H * v_dim] (any row stride): the result is multiplied by sigmoid(gate), last."""
     t = q.shape[0]
     hq, d = num_q_heads, head_dim
     dv = d if v_dim is None else v_dim
@@ -545,6 +553,9 @@ def window_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
             att = softcap * torch.tanh(att / softcap)
         qi = torch.arange(ql, device=q.device).view(ql, 1) + (sl[s] - ql)
         kj = torch.arange(sl[s], device=q.device).view(1, sl[s])
+        if dist_bias is not None:
+            r1, r2 = (r.float().view(hq, 1, 1) for r in dist_bias)
+            att = att - r1 * torch.log1p(r2 * (qi - kj).clamp(min=0).unsqueeze(0))
         dead = kj > qi
         if window is not None:
             dead = dead | (qi - kj >= window)
@@ -554,7 +565,15 @@ def window_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         if sink is not None:
             att = torch.cat([att, sink.float().view(hq, 1, 1).expand(hq, ql, 1)], dim=-1)
         p = torch.softmax(att, dim=-1)[..., : sl[s]]
-        out[q0:q1] = (torch.einsum("hqk,khd->qhd", p, vv).reshape(ql, hq * dv) * out_scale).to(q.dtype)
+        o = torch.einsum("hqk,khd->qhd", p, vv)
+        if v_turn is not None:
+            c, sn = v_turn[q0:q1, None, :dv // 2], v_turn[q0:q1, None, dv // 2:]
+            a, b = o[..., :dv // 2], o[..., dv // 2:]
+            o = torch.cat([a * c + b * sn, b * c - a * sn], -1)
+        o = o.reshape(ql, hq * dv) * out_scale
+        if gate is not None:
+            o = o * torch.sigmoid(gate[q0:q1].float())
+        out[q0:q1] = o.to(q.dtype)
     return out
 
 
@@ -663,16 +682,49 @@ def rotate_half_pairs(x: torch.Tensor, positions: torch.Tensor, rot_dims: int, b
     return torch.cat([a * c - b * s, b * c + a * s, x[..., rot_dims:]], -1)
 
 
+def rotary_angles(positions: torch.Tensor, freqs: torch.Tensor) -> torch.Tensor:
+    """[T, 2 n] fp32: cos, then sin, of position * freqs[i] (fp64 frequencies, angles formed in fp64)."""
+    a = positions.double()[:, None] * freqs.double()[None, :]
+    return torch.cat([torch.cos(a), torch.sin(a)], -1).float()
+
+
+def turn_pairs(x: torch.Tensor, angles: Optional[torch.Tensor]) -> torch.Tensor:
+    """x [T, heads, d] fp32; entry i < n turns with entry i + n by the row's angle i (n = angles' width / 2)."""
+    if angles is None or angles.shape[1] == 0:
+        return x
+    n = angles.shape[1] // 2
+    c, s = angles[:, None, :n], angles[:, None, n:]
+    u, v = x[..., :n], x[..., n:2 * n]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * n:]], -1)
+
+
 def qk_norm_rope_kv_write(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, dim: int, v_dim: int, q_norm_w,
                           k_norm_w, eps: float, positions: torch.Tensor, rot_dims: int, rot_base: float,
                           k_cache: torch.Tensor, v_cache: torch.Tensor, slots: torch.Tensor,
-                          freqs: Optional[torch.Tensor] = None, mag: float = 1.0) -> torch.Tensor:
+                          freqs: Optional[torch.Tensor] = None, mag: float = 1.0, unit_norm: bool = False,
+                          angles: Optional[torch.Tensor] = None,
+                          v_angles: Optional[torch.Tensor] = None) -> torch.Tensor:
     """qkv [T, >= H*D + G*D + G*Dv] = [queries | keys | values]. Per-head RMS norm of q and k (weights optional),
     then the rotate-half rotation of both; rotated keys go to the K cache, values as projected to the V cache.
     Returns the queries [T, H * D]. With num_kv_heads == 0 the row holds queries only (a layer that reads another
-    layer's keys and values) and no cache is touched. `freqs`, `mag`: see `rotate_half_pairs`."""
+    layer's keys and values) and no cache is touched. `freqs`, `mag`: see `rotate_half_pairs`. `unit_norm`: q and k
+    are divided by their root mean square per head without a weight. `angles` [T, rot_dims] fp32 (cos | sin per pair,
+    see `rotary_angles`) replaces the base / frequencies; `v_angles` [T, v_dim] likewise: the values are rotated too,
+    over their whole width, and cached so."""
     t = qkv.shape[0]
     hd, gd = num_heads * dim, num_kv_heads * dim
+    if unit_norm:
+        q_norm_w = k_norm_w = torch.ones(dim, device=qkv.device)
+    if angles is not None or v_angles is not None:
+        assert num_kv_heads > 0
+        q, k = (qkv[:, a:b].reshape(t, -1, dim).float() for a, b in ((0, hd), (hd, hd + gd)))
+        v = qkv[:, hd + gd:hd + gd + num_kv_heads * v_dim].reshape(t, num_kv_heads, v_dim)
+        if q_norm_w is not None:
+            q = q * torch.rsqrt((q * q).mean(-1, keepdim=True) + eps) * q_norm_w.float()
+            k = k * torch.rsqrt((k * k).mean(-1, keepdim=True) + eps) * k_norm_w.float()
+        _cache_rows_write(k_cache, slots, turn_pairs(k, angles).to(qkv.dtype))
+        _cache_rows_write(v_cache, slots, turn_pairs(v.float(), v_angles).to(qkv.dtype))
+        return turn_pairs(q, angles).to(qkv.dtype).reshape(t, hd)
     q = qkv[:, :hd].reshape(t, num_heads, dim).float()
     if num_kv_heads == 0:
         if q_norm_w is not None:
@@ -767,6 +819,58 @@ def gated_group_norm(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, group
     return out
 
 
+def gate_then_norm(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, group: int, eps: float,
+                   out: Optional[torch.Tensor] = None, out_dtype=None) -> torch.Tensor:
+    """v = o * silu(gate) [T, n], RMS norm over consecutive groups of `group` columns, times w [n] (fp32)."""
+    t, n = o.shape
+    x = (o.float() * F.silu(gate.float())).reshape(t, n // group, group)
+    x = (x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps)).reshape(t, n) * w.float()
+    if out is None:
+        return x.to(out_dtype or gate.dtype)
+    out.copy_(x.to(out.dtype))
+    return out
+
+
+def ssd_scan(x: torch.Tensor, b: torch.Tensor, c: torch.Tensor, dt: torch.Tensor, neg_a: torch.Tensor,
+             dt_bias: torch.Tensor, d_skip: torch.Tensor, state: Optional[torch.Tensor], rec_slots, seq_lens,
+             query_start_loc, heads: int, groups: int, nstate: int, v_dim: int) -> torch.Tensor:
+    """Mamba-2 recurrence per head, fp32, token by token, S [nstate, v_dim] (head h reads group h // (heads / groups)
+    of b and c): dt = softplus(dt + dt_bias[h]);  S <- exp(neg_a[h] dt) S + dt b x^T;  y = S^T c + d_skip[h] x.
+    x [T, heads * v_dim], b / c [T, groups * nstate], dt [T, heads]; state [slots, heads, nstate, v_dim] fp32 carries S
+    between portions (zeros for one that starts at position 0). -> y [T, heads * v_dim] fp32."""
+    t = x.shape[0]
+    out = torch.zeros(t, heads * v_dim, dtype=torch.float32, device=x.device)
+    qsl, sl = query_start_loc.tolist(), seq_lens.tolist()
+    rep = heads // groups
+    for s in range(len(sl)):
+        q0, q1 = qsl[s], qsl[s + 1]
+        n = q1 - q0
+        if n <= 0:
+            continue
+        xx = x[q0:q1].float().reshape(n, heads, v_dim)
+        bb = b[q0:q1].float().reshape(n, groups, nstate).repeat_interleave(rep, 1)
+        cc = c[q0:q1].float().reshape(n, groups, nstate).repeat_interleave(rep, 1)
+        step = F.softplus(dt[q0:q1].float() + dt_bias.float(), threshold=80.0)
+        g = torch.exp(neg_a.float() * step)
+        st = torch.zeros(heads, nstate, v_dim, dtype=torch.float32, device=x.device)
+        if state is not None and sl[s] - n > 0:
+            st = state[int(rec_slots[s])].clone()
+        y = torch.empty(n, heads, v_dim, dtype=torch.float32, device=x.device)
+        for i in range(n):
+            st = st * g[i].view(heads, 1, 1) + bb[i].unsqueeze(-1) * (step[i].view(heads, 1) * xx[i]).unsqueeze(1)
+            y[i] = torch.einsum("hnv,hn->hv", st, cc[i]) + d_skip.float().view(heads, 1) * xx[i]
+        out[q0:q1] = y.reshape(n, heads * v_dim)
+        if state is not None:
+            state[int(rec_slots[s])] = st
+    return out
+
+
+def gelu_gate_embed(g: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, col0: int) -> torch.Tensor:
+    """gelu_tanh(g) * table[ids, col0 : col0 + dim] for g [T, dim]."""
+    e = table[ids.long(), col0:col0 + g.shape[1]]
+    return (F.gelu(g.float(), approximate="tanh") * e.float()).to(g.dtype)
+
+
 def silu_mul(gu: torch.Tensor) -> torch.Tensor:
     """gu [T, 2F] = [gate | up] -> silu(gate) * up."""
     f = gu.shape[1] // 2
@@ -857,6 +961,22 @@ def pair_rotary_frequencies(dims: int, base: float, scaling: Optional[dict] = No
         f = f / factor * ramp + f * (1.0 - ramp)
         mag = 0.1 * math.log(factor) + 1.0
     return f.to(dtype), float(mag)
+
+
+def banded_rotary_frequencies(dims: int, base: float, scaling: Optional[dict] = None,
+                              dtype=torch.float64) -> torch.Tensor:
+    """Frequency per pair with Llama 3.1 style `scaling` {factor, low, high, original}: by wavelength 2 pi / f, short
+    waves (< original / high) keep f, long ones (> original / low) take f / factor, those between are blended by
+    s = (original / wavelength - low) / (high - low): (1 - s) f / factor + s f."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = torch.exp(-(2.0 * i / max(dims, 1)) * math.log(base))
+    if scaling:
+        factor, low, high, orig = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
+        wave = 2.0 * math.pi / f
+        s = (orig / wave - low) / (high - low) if high != low else torch.zeros_like(f)
+        mid = (1.0 - s) * f / factor + s * f
+        f = torch.where(wave < orig / high, f, torch.where(wave > orig / low, f / factor, mid))
+    return f.to(dtype)
 
 
 def rotate_adjacent_pairs(x: torch.Tensor, positions: torch.Tensor, freqs: torch.Tensor, mag: float) -> torch.Tensor:
