@@ -89,4 +89,33 @@ inline int get_kv_tmap(const void* base, int64_t num_pages, int Hkv, int D, int 
 // |error| ~ 1e-7 near 0
 __device__ __forceinline__ float tanh_exp(float x) { return 1.0f - __fdividef(2.0f, __expf(2.0f * x) + 1.0f); }
 
+// Options that some designs add to the masked attention (all of them optional):
+//   r1, r2 [Hq]     distance bias: r1 ln(1 + r2 (i - j)) is taken off the scaled score of key j for the query at i
+//   v_turn [tok, D] cos | sin (fp32) of the query's position: the values were rotated by their own positions, every
+//                   head's result is turned back by the query's (entry m with m + D / 2)
+//   gate            [tok, Hq * D] rows of stride ldg: the result is multiplied by sigmoid(gate), last
+struct AttnExtras {
+  const float* r1 = nullptr;
+  const float* r2 = nullptr;
+  const __nv_bfloat16* gate = nullptr;
+  int64_t ldg = 0;
+  const float* v_turn = nullptr;
+  bool any() const { return r1 != nullptr || gate != nullptr || v_turn != nullptr; }
+};
+inline AttnExtras make_extras(const void* r1, const void* r2, const void* gate, int64_t ldg, const void* v_turn) {
+  AttnExtras e;
+  e.r1 = reinterpret_cast<const float*>(r1);
+  e.r2 = reinterpret_cast<const float*>(r2);
+  e.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  e.ldg = ldg;
+  e.v_turn = reinterpret_cast<const float*>(v_turn);
+  return e;
+}
+
+// the distance bias in the base-2 domain of the softmax: r1 ln(.) log2(e) = r1 log2(.)
+__device__ __forceinline__ float dist_bias_log2(float r1, float r2, int dist) {
+  return r1 * __log2f(fmaf(r2, (float)max(dist, 0), 1.0f));
+}
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
+
 }  // namespace b200

@@ -47,6 +47,7 @@ struct AttnParams {
   // score cap (cap_log2 > 0): a scaled score s becomes cap * tanh(s / cap) before the mask and the softmax;
   // scale_over_cap = scale / cap, cap_log2 = cap * log2(e)
   float cap_log2, scale_over_cap;
+  AttnExtras ex;      // distance bias, turned values, output gate (num_splits == 1)
 };
 
 
@@ -91,7 +92,7 @@ __device__ __forceinline__ void kv_producer(const CUtensorMap* tk, const CUtenso
 // ---------------------------------------------------------------------------------------------
 // decode kernel
 // ---------------------------------------------------------------------------------------------
-template <int D>
+template <int D, bool EX>
 __global__ void __launch_bounds__(kAttnThreads)
 attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v,
                    const AttnParams p) {
@@ -156,6 +157,12 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_cons
   for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY};
   float l_run[2] = {0.f, 0.f};
+  float b1[2] = {0.f, 0.f}, b2[2] = {0.f, 0.f};      // distance bias of this thread's two heads
+  if (EX && p.ex.r1 != nullptr) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+      if (g + 8 * r < p.GP) { b1[r] = p.ex.r1[hbase + g + 8 * r]; b2[r] = p.ex.r2[hbase + g + 8 * r]; }
+  }
 
   uint32_t it = 0;
   for (int tile = tile_begin; tile < tile_end; ++tile, ++it) {
@@ -191,6 +198,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_cons
       for (int e = 0; e < 4; ++e) {
         const int col = abs0 + nt * 8 + (e & 1);
         float v = p.cap_log2 > 0.f ? p.cap_log2 * tanh_exp(sc[nt][e] * p.scale_over_cap) : sc[nt][e] * p.scale_log2;
+        if (EX) v -= dist_bias_log2(b1[e >> 1], b2[e >> 1], seq_len - 1 - col);
         if (col >= seq_len || col < win_lo) v = -INFINITY;
         sc[nt][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -289,7 +297,27 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_cons
         const float4 v = *reinterpret_cast<const float4*>(red_o + (w * 16 + row) * D + c);
         acc.x += wgt[w] * v.x; acc.y += wgt[w] * v.y; acc.z += wgt[w] * v.z; acc.w += wgt[w] * v.w;
       }
+      if (EX && p.ex.v_turn != nullptr) {
+        const int cp = c < D / 2 ? c + D / 2 : c - D / 2;
+        float4 oth = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int w = 0; w < kMathWarps; ++w) {
+          const float4 v = *reinterpret_cast<const float4*>(red_o + (w * 16 + row) * D + cp);
+          oth.x += wgt[w] * v.x; oth.y += wgt[w] * v.y; oth.z += wgt[w] * v.z; oth.w += wgt[w] * v.w;
+        }
+        const float* tr = p.ex.v_turn + (size_t)seq * D + (c < D / 2 ? c : cp);
+        const float4 cs = *reinterpret_cast<const float4*>(tr), sn = *reinterpret_cast<const float4*>(tr + D / 2);
+        const float sg = c < D / 2 ? 1.f : -1.f;
+        acc.x = acc.x * cs.x + sg * oth.x * sn.x; acc.y = acc.y * cs.y + sg * oth.y * sn.y;
+        acc.z = acc.z * cs.z + sg * oth.z * sn.z; acc.w = acc.w * cs.w + sg * oth.w * sn.w;
+      }
       acc.x *= inv; acc.y *= inv; acc.z *= inv; acc.w *= inv;
+      if (EX && p.ex.gate != nullptr) {
+        const uint2 gv = *reinterpret_cast<const uint2*>(p.ex.gate + (size_t)seq * p.ex.ldg + (size_t)head * D + c);
+        const float2 g0 = unpack_bf16(gv.x), g1 = unpack_bf16(gv.y);
+        acc.x *= sigmoid_fast(g0.x); acc.y *= sigmoid_fast(g0.y);
+        acc.z *= sigmoid_fast(g1.x); acc.w *= sigmoid_fast(g1.y);
+      }
       if (p.num_splits == 1) {
         uint2 ov = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
         *reinterpret_cast<uint2*>(p.out + (size_t)seq * p.out_ts + (size_t)head * D + c) = ov;
@@ -369,7 +397,7 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
 // ---------------------------------------------------------------------------------------------
 // prefill kernel: 64 rows = (64 / GP) tokens x GP heads, warps split rows
 // ---------------------------------------------------------------------------------------------
-template <int D>
+template <int D, bool EX>
 __global__ void __launch_bounds__(kAttnThreads)
 attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v,
                     const AttnParams p) {
@@ -447,6 +475,11 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
   const int lim[2] = {ctx_len + r_tok[0], ctx_len + r_tok[1]};  // last visible key per row
   const int clo[2] = {p.chunk > 0 ? (max(lim[0], 0) / p.chunk) * p.chunk : 0,
                       p.chunk > 0 ? (max(lim[1], 0) / p.chunk) * p.chunk : 0};   // first key of the row's chunk
+  float b1[2] = {0.f, 0.f}, b2[2] = {0.f, 0.f};      // distance bias of this thread's two rows
+  if (EX && p.ex.r1 != nullptr) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) { b1[r] = p.ex.r1[r_head[r]]; b2[r] = p.ex.r2[r_head[r]]; }
+  }
 
   uint32_t it = 0;
   for (int tile = tile_lo; tile < n_tiles; ++tile, ++it) {
@@ -479,6 +512,7 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
       for (int e = 0; e < 4; ++e) {
         const int col = abs0 + nt * 8 + (e & 1);
         float v = p.cap_log2 > 0.f ? p.cap_log2 * tanh_exp(sc[nt][e] * p.scale_over_cap) : sc[nt][e] * p.scale_log2;
+        if (EX) v -= dist_bias_log2(b1[e >> 1], b2[e >> 1], lim[e >> 1] - col);
         if (col > lim[e >> 1] || col < clo[e >> 1] || (p.window > 0 && col <= lim[e >> 1] - p.window)) v = -INFINITY;
         sc[nt][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -543,6 +577,29 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
     if (p.sink != nullptr && m_run[r] > -INFINITY) den += exp2f(p.sink[r_head[r]] * 1.4426950408889634f - m_run[r]);
     const float inv = (den > 0.f ? 1.f / den : 0.f) * p.out_scale;
     __nv_bfloat16* op = p.out + (size_t)(q_begin + r_tok[r]) * p.out_ts + (size_t)r_head[r] * D + 2 * t;
+    if (EX && p.ex.v_turn != nullptr) {              // entry m and m + D / 2 are n-tiles nd and nd + D / 16
+      const float* tr = p.ex.v_turn + (size_t)(q_begin + r_tok[r]) * D + 2 * t;
+#pragma unroll
+      for (int nd = 0; nd < D / 16; ++nd) {
+        const float2 cs = *reinterpret_cast<const float2*>(tr + nd * 8);
+        const float2 sn = *reinterpret_cast<const float2*>(tr + D / 2 + nd * 8);
+        const float u0 = o[nd][2 * r], u1 = o[nd][2 * r + 1];
+        const float v0 = o[nd + D / 16][2 * r], v1 = o[nd + D / 16][2 * r + 1];
+        o[nd][2 * r] = u0 * cs.x + v0 * sn.x;
+        o[nd][2 * r + 1] = u1 * cs.y + v1 * sn.y;
+        o[nd + D / 16][2 * r] = v0 * cs.x - u0 * sn.x;
+        o[nd + D / 16][2 * r + 1] = v1 * cs.y - u1 * sn.y;
+      }
+    }
+    if (EX && p.ex.gate != nullptr) {
+      const __nv_bfloat16* gp = p.ex.gate + (size_t)(q_begin + r_tok[r]) * p.ex.ldg + (size_t)r_head[r] * D + 2 * t;
+#pragma unroll
+      for (int nd = 0; nd < D / 8; ++nd) {
+        const float2 gv = unpack_bf16(*reinterpret_cast<const uint32_t*>(gp + nd * 8));
+        o[nd][2 * r] *= sigmoid_fast(gv.x);
+        o[nd][2 * r + 1] *= sigmoid_fast(gv.y);
+      }
+    }
 #pragma unroll
     for (int nd = 0; nd < D / 8; ++nd) {
       *reinterpret_cast<uint32_t*>(op + nd * 8) = pack_bf16(o[nd][2 * r] * inv, o[nd][2 * r + 1] * inv);
@@ -568,32 +625,32 @@ static int largest_divisor_leq(int G, int cap, int must_divide) {
   return 1;
 }
 
-template <int D>
+template <int D, bool EX>
 static int launch_decode(const CUtensorMap& tk, const CUtensorMap& tv, const AttnParams& p, int num_seqs,
                          cudaStream_t st) {
   using SM = AttnSmem<D>;
   static PerDeviceOnce configured;
   if (configured.need()) {
-    CUDA_CHECK_RET(cudaFuncSetAttribute(attn_decode_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, SM::kBytes));
+    CUDA_CHECK_RET(cudaFuncSetAttribute(attn_decode_kernel<D, EX>, cudaFuncAttributeMaxDynamicSharedMemorySize, SM::kBytes));
     configured.done();
   }
   dim3 grid(p.Hkv * (p.G / p.GP), num_seqs, p.num_splits);
-  CUDA_CHECK_RET(launch_pdl(attn_decode_kernel<D>, grid, dim3(kAttnThreads), SM::kBytes, st, tk, tv, p));
+  CUDA_CHECK_RET(launch_pdl(attn_decode_kernel<D, EX>, grid, dim3(kAttnThreads), SM::kBytes, st, tk, tv, p));
   return 0;
 }
 
-template <int D>
+template <int D, bool EX>
 static int launch_prefill(const CUtensorMap& tk, const CUtensorMap& tv, const AttnParams& p, int num_seqs,
                           int max_q_len, cudaStream_t st) {
   using SM = AttnSmem<D>;
   static PerDeviceOnce configured;
   if (configured.need()) {
-    CUDA_CHECK_RET(cudaFuncSetAttribute(attn_prefill_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, SM::kBytes));
+    CUDA_CHECK_RET(cudaFuncSetAttribute(attn_prefill_kernel<D, EX>, cudaFuncAttributeMaxDynamicSharedMemorySize, SM::kBytes));
     configured.done();
   }
   const int toks_per_tile = 64 / p.GP;
   dim3 grid((max_q_len + toks_per_tile - 1) / toks_per_tile, num_seqs, p.Hkv * (p.G / p.GP));
-  attn_prefill_kernel<D><<<grid, kAttnThreads, SM::kBytes, st>>>(tk, tv, p);
+  attn_prefill_kernel<D, EX><<<grid, kAttnThreads, SM::kBytes, st>>>(tk, tv, p);
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
 }
@@ -609,7 +666,11 @@ static int attn_decode_impl(const void* q, int64_t q_ts, void* out, const void* 
                             void* part_lse, int num_seqs, int seq_offset, int max_blocks, int Hq, int Hkv,
                             int D, int page_size, int num_splits, float scale, void* split_cnt, void* stream,
                             int window, const void* sink, int chunk = 0, int64_t out_ts = 0, float out_scale = 1.0f,
-                            float softcap = 0.0f) {
+                            float softcap = 0.0f, const AttnExtras& ex = AttnExtras()) {
+  if (ex.any() && num_splits > 1) {
+    fprintf(stderr, "[gllm_b200] attn_decode: distance bias, turned values and gate need num_splits == 1\n");
+    return 1;
+  }
   if (softcap > 0.f && num_splits > 1) {
     fprintf(stderr, "[gllm_b200] attn_decode: a score cap needs num_splits == 1\n");
     return 1;
@@ -627,6 +688,7 @@ static int attn_decode_impl(const void* q, int64_t q_ts, void* out, const void* 
   if (get_kv_tmap(k_cache, num_pages, Hkv, D, page_size, &tk)) return 1;
   if (get_kv_tmap(v_cache, num_pages, Hkv, D, page_size, &tv)) return 1;
   AttnParams p;
+  p.ex = ex;
   p.q = reinterpret_cast<const __nv_bfloat16*>(q); p.q_ts = q_ts;
   p.out = reinterpret_cast<__nv_bfloat16*>(out);
   p.part_o = reinterpret_cast<float*>(part_o);
@@ -651,9 +713,15 @@ static int attn_decode_impl(const void* q, int64_t q_ts, void* out, const void* 
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   int rc;
   switch (D) {
-    case 64: rc = launch_decode<64>(tk, tv, p, num_seqs, st); break;
-    case 128: rc = launch_decode<128>(tk, tv, p, num_seqs, st); break;
-    case 256: rc = launch_decode<256>(tk, tv, p, num_seqs, st); break;
+    case 64: rc = p.ex.any() ? launch_decode<64, true>(tk, tv, p, num_seqs, st)
+                            : launch_decode<64, false>(tk, tv, p, num_seqs, st);
+      break;
+    case 128: rc = p.ex.any() ? launch_decode<128, true>(tk, tv, p, num_seqs, st)
+                            : launch_decode<128, false>(tk, tv, p, num_seqs, st);
+      break;
+    case 256: rc = p.ex.any() ? launch_decode<256, true>(tk, tv, p, num_seqs, st)
+                            : launch_decode<256, false>(tk, tv, p, num_seqs, st);
+      break;
     default:
       fprintf(stderr, "[gllm_b200] attn_decode: unsupported head_dim %d\n", D);
       return 1;
@@ -695,7 +763,7 @@ static int attn_prefill_impl(const void* q, int64_t q_ts, void* out, const void*
                              const void* q_start, int num_seqs, int seq_offset, int max_q_len, int max_blocks,
                              int Hq, int Hkv, int D, int page_size, float scale, void* stream, int window,
                              const void* sink, int chunk = 0, int64_t out_ts = 0, float out_scale = 1.0f,
-                             float softcap = 0.0f) {
+                             float softcap = 0.0f, const AttnExtras& ex = AttnExtras()) {
   if (num_seqs <= 0 || max_q_len <= 0) return 0;
   if (page_size < 8 || kTileN % page_size != 0 || Hq % Hkv != 0) {
     fprintf(stderr, "[gllm_b200] attn_prefill: unsupported page_size=%d / heads\n", page_size);
@@ -705,6 +773,7 @@ static int attn_prefill_impl(const void* q, int64_t q_ts, void* out, const void*
   if (get_kv_tmap(k_cache, num_pages, Hkv, D, page_size, &tk)) return 1;
   if (get_kv_tmap(v_cache, num_pages, Hkv, D, page_size, &tv)) return 1;
   AttnParams p;
+  p.ex = ex;
   p.q = reinterpret_cast<const __nv_bfloat16*>(q); p.q_ts = q_ts;
   p.out = reinterpret_cast<__nv_bfloat16*>(out);
   p.part_o = nullptr; p.part_lse = nullptr;
@@ -721,9 +790,12 @@ static int attn_prefill_impl(const void* q, int64_t q_ts, void* out, const void*
   p.scale_over_cap = softcap > 0.f ? scale / softcap : 0.f;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   switch (D) {
-    case 64: return launch_prefill<64>(tk, tv, p, num_seqs, max_q_len, st);
-    case 128: return launch_prefill<128>(tk, tv, p, num_seqs, max_q_len, st);
-    case 256: return launch_prefill<256>(tk, tv, p, num_seqs, max_q_len, st);
+    case 64: return p.ex.any() ? launch_prefill<64, true>(tk, tv, p, num_seqs, max_q_len, st)
+                               : launch_prefill<64, false>(tk, tv, p, num_seqs, max_q_len, st);
+    case 128: return p.ex.any() ? launch_prefill<128, true>(tk, tv, p, num_seqs, max_q_len, st)
+                               : launch_prefill<128, false>(tk, tv, p, num_seqs, max_q_len, st);
+    case 256: return p.ex.any() ? launch_prefill<256, true>(tk, tv, p, num_seqs, max_q_len, st)
+                               : launch_prefill<256, false>(tk, tv, p, num_seqs, max_q_len, st);
     default:
       fprintf(stderr, "[gllm_b200] attn_prefill: unsupported head_dim %d\n", D);
       return 1;
@@ -752,10 +824,12 @@ GLLM_EXPORT int gllm_attn_decode_mask(const void* q, int64_t q_ts, void* out, in
                                       const void* v_cache, int64_t num_pages, const void* block_table,
                                       const void* seq_lens, int num_seqs, int seq_offset, int max_blocks, int Hq,
                                       int Hkv, int D, int page_size, float scale, int window, int chunk,
-                                      const void* sink, float out_scale, float softcap, void* stream) {
+                                      const void* sink, float out_scale, float softcap, const void* r1,
+                                      const void* r2, const void* gate, int64_t ldg, const void* v_turn,
+                                      void* stream) {
   return attn_decode_impl(q, q_ts, out, k_cache, v_cache, num_pages, block_table, seq_lens, nullptr, nullptr,
                           num_seqs, seq_offset, max_blocks, Hq, Hkv, D, page_size, 1, scale, nullptr, stream, window,
-                          sink, chunk, out_ts, out_scale, softcap);
+                          sink, chunk, out_ts, out_scale, softcap, make_extras(r1, r2, gate, ldg, v_turn));
 }
 
 GLLM_EXPORT int gllm_attn_prefill_mask(const void* q, int64_t q_ts, void* out, int64_t out_ts, const void* k_cache,
@@ -763,8 +837,9 @@ GLLM_EXPORT int gllm_attn_prefill_mask(const void* q, int64_t q_ts, void* out, i
                                        const void* seq_lens, const void* q_start, int num_seqs, int seq_offset,
                                        int max_q_len, int max_blocks, int Hq, int Hkv, int D, int page_size,
                                        float scale, int window, int chunk, const void* sink, float out_scale,
-                                       float softcap, void* stream) {
+                                       float softcap, const void* r1, const void* r2, const void* gate, int64_t ldg,
+                                       const void* v_turn, void* stream) {
   return attn_prefill_impl(q, q_ts, out, k_cache, v_cache, num_pages, block_table, seq_lens, q_start, num_seqs,
                            seq_offset, max_q_len, max_blocks, Hq, Hkv, D, page_size, scale, stream, window, sink,
-                           chunk, out_ts, out_scale, softcap);
+                           chunk, out_ts, out_scale, softcap, make_extras(r1, r2, gate, ldg, v_turn));
 }

@@ -48,6 +48,9 @@ struct TcAttnParams {
   // value (null = none)
   float cap_log2, scale_over_cap;
   const float* sink;
+  int64_t out_ts;     // output row stride (elements)
+  int window;         // sliding window: a query at i sees keys j with i - j < window (0 = the whole past)
+  AttnExtras ex;      // distance bias (kernel template BIAS), turned values, output gate
   uint32_t v_lbo16, v_sbo16, v_kadv16, v_split_n;   // MN-major V descriptor fields (16-byte units)
 };
 
@@ -98,7 +101,7 @@ __device__ __forceinline__ uint32_t a_tile_off(int row, int c) {
   return (c >> 3) * (kTcRows * 128) + row * 128 + (((c & 7) ^ (row & 7)) << 4);
 }
 
-template <int D, int KV, bool CAP>
+template <int D, int KV, bool CAP, bool BIAS>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v,
                        const TcAttnParams p) {
@@ -132,7 +135,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
   const int ctx_len = seq_len - q_len;
   const int last_tok = min(tok_base + toks_per_tile, q_len) - 1;
   const int kv_end = ctx_len + last_tok + 1;           // causal horizon of this tile
-  const int n_tiles = (kv_end + KV - 1) / KV;
+  // KV tiles [tile0, tile0 + n_tiles): with a window the first query's oldest visible key decides where they start;
+  // pipeline indices (stages, phases, buffers) count from 0
+  const int tile0 = p.window > 0 ? max(0, ctx_len + tok_base - p.window + 1) / KV : 0;
+  const int n_tiles = (kv_end + KV - 1) / KV - tile0;
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < SM::kStages; ++i) {
@@ -169,7 +175,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
         uint8_t* sv = sk + SM::kTileBytes;
         mbar_expect_tx(&kv_full[s], SM::kStageBytes);
         for (int j = 0; j < pages_per_tile; ++j) {
-          int pi = tile * pages_per_tile + j;
+          int pi = (tile0 + tile) * pages_per_tile + j;
           if (pi > last_page) pi = last_page;          // masked columns: keep the data finite
           const int slab0 = (bt[pi] * p.Hkv + kvh) * (D / 64);
 #pragma unroll
@@ -256,14 +262,19 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
       mbar_arrive(q_full);
     }
     const int lim = ctx_len + tok;                       // last visible key of this row
+    const int low = p.window > 0 ? lim - p.window + 1 : 0;          // first visible key of this row
+    float b1 = 0.f, b2 = 0.f;
+    if (BIAS) { b1 = p.ex.r1[head]; b2 = p.ex.r2[head]; }
     float m_run = -INFINITY, l_run = 0.f;
     for (int tile = 0; tile < n_tiles; ++tile) {
       const int b = tile & 1;
       mbar_wait(&s_full[b], (tile >> 1) & 1);
       tc_fence_after();
       const uint32_t t_s = tmem + lane_base + b * KV;
-      const int key0 = tile * KV;
-      const bool need_mask = key0 + KV - 1 > ctx_len + tok_base;   // CTA-uniform: a diagonal tile
+      const int key0 = (tile0 + tile) * KV;
+      // CTA-uniform: a diagonal tile, or one that the window of some row starts in
+      const bool need_mask = key0 + KV - 1 > ctx_len + tok_base ||
+                             (p.window > 0 && key0 < ctx_len + last_tok - p.window + 1);
       // pass 1: row max
       float mx = -INFINITY;
 #pragma unroll 1
@@ -271,16 +282,24 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
         uint32_t v[32];
         tmem_ld_32x32(t_s + c, v);
         tmem_ld_wait();
-        if (need_mask) {
+        if (BIAS) {
 #pragma unroll
-          for (int e = 0; e < 32; ++e) mx = fmaxf(mx, (key0 + c + e <= lim) ? __uint_as_float(v[e]) : -INFINITY);
+          for (int e = 0; e < 32; ++e) {
+            const int key = key0 + c + e;
+            const float x = fmaf(__uint_as_float(v[e]), p.scale_log2, -dist_bias_log2(b1, b2, lim - key));
+            mx = fmaxf(mx, (key <= lim && key >= low) ? x : -INFINITY);
+          }
+        } else if (need_mask) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e)
+            mx = fmaxf(mx, (key0 + c + e <= lim && key0 + c + e >= low) ? __uint_as_float(v[e]) : -INFINITY);
         } else {
 #pragma unroll
           for (int e = 0; e < 32; ++e) mx = fmaxf(mx, __uint_as_float(v[e]));
         }
       }
       // the cap is increasing in the score: the capped maximum is the cap of the raw maximum
-      const float mx_s = !CAP ? mx * p.scale_log2
+      const float mx_s = BIAS ? mx : !CAP ? mx * p.scale_log2
                               : (mx == -INFINITY ? -INFINITY : p.cap_log2 * tanh_exp(mx * p.scale_over_cap));
       const float m_new = fmaxf(m_run, mx_s);
       const float m_use = (m_new == -INFINITY) ? 0.f : m_new;
@@ -297,9 +316,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
         float f[32];
 #pragma unroll
         for (int e = 0; e < 32; ++e) {
-          float x = CAP ? exp2f(fmaf(p.cap_log2, tanh_exp(__uint_as_float(v[e]) * p.scale_over_cap), -m_use))
+          float x = BIAS ? exp2f(fmaf(__uint_as_float(v[e]), p.scale_log2,
+                                      -dist_bias_log2(b1, b2, lim - (key0 + c + e)) - m_use))
+                    : CAP ? exp2f(fmaf(p.cap_log2, tanh_exp(__uint_as_float(v[e]) * p.scale_over_cap), -m_use))
                         : exp2f(fmaf(__uint_as_float(v[e]), p.scale_log2, -m_use));
-          if (need_mask && key0 + c + e > lim) x = 0.f;
+          if (need_mask && (key0 + c + e > lim || key0 + c + e < low)) x = 0.f;
           f[e] = x;
           sum += x;
         }
@@ -343,22 +364,73 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
     tc_fence_after();
     if (p.sink != nullptr && row_ok && m_run > -INFINITY) l_run += exp2f(p.sink[head] * 1.4426950408889634f - m_run);
     const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-    __nv_bfloat16* op = p.out + (static_cast<size_t>(q_begin + tok) * p.Hq + head) * D;
+    __nv_bfloat16* op = p.out + static_cast<size_t>(q_begin + tok) * p.out_ts + static_cast<size_t>(head) * D;
+    const __nv_bfloat16* gp = p.ex.gate != nullptr && row_ok
+                                  ? p.ex.gate + static_cast<size_t>(q_begin + tok) * p.ex.ldg + static_cast<size_t>(head) * D
+                                  : nullptr;
     const uint32_t t_o = tmem_o + lane_base;
-#pragma unroll 1
-    for (int c = 0; c < D; c += 32) {
-      uint32_t v[32];
-      tmem_ld_32x32(t_o + c, v);
-      tmem_ld_wait();
-      if (row_ok) {
+    // 32 finished columns from column c on: normalise, gate, round, store
+    auto store32 = [&](int c, const float (&f)[32]) {
 #pragma unroll
-        for (int g = 0; g < 4; ++g) {
-          uint4 w;
-          w.x = pack_bf16(__uint_as_float(v[g * 8 + 0]) * inv, __uint_as_float(v[g * 8 + 1]) * inv);
-          w.y = pack_bf16(__uint_as_float(v[g * 8 + 2]) * inv, __uint_as_float(v[g * 8 + 3]) * inv);
-          w.z = pack_bf16(__uint_as_float(v[g * 8 + 4]) * inv, __uint_as_float(v[g * 8 + 5]) * inv);
-          w.w = pack_bf16(__uint_as_float(v[g * 8 + 6]) * inv, __uint_as_float(v[g * 8 + 7]) * inv);
-          *reinterpret_cast<uint4*>(op + c + g * 8) = w;
+      for (int g = 0; g < 4; ++g) {
+        float x[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = f[g * 8 + e] * inv;
+        if (gp != nullptr) {
+          const uint4 gv = *reinterpret_cast<const uint4*>(gp + c + g * 8);
+          const uint32_t gw[4] = {gv.x, gv.y, gv.z, gv.w};
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float2 z = unpack_bf16(gw[e]);
+            x[2 * e] *= sigmoid_fast(z.x);
+            x[2 * e + 1] *= sigmoid_fast(z.y);
+          }
+        }
+        uint4 w;
+        w.x = pack_bf16(x[0], x[1]);
+        w.y = pack_bf16(x[2], x[3]);
+        w.z = pack_bf16(x[4], x[5]);
+        w.w = pack_bf16(x[6], x[7]);
+        *reinterpret_cast<uint4*>(op + c + g * 8) = w;
+      }
+    };
+    if (p.ex.v_turn != nullptr) {
+      // turn the head's result back: columns m and m + D / 2 of this row, both in this thread's TMEM lane
+      const float4* tr = reinterpret_cast<const float4*>(p.ex.v_turn + static_cast<size_t>(q_begin + (row_ok ? tok : 0)) * D);
+#pragma unroll 1
+      for (int c = 0; c < D / 2; c += 32) {
+        uint32_t a[32], b[32];
+        tmem_ld_32x32(t_o + c, a);
+        tmem_ld_32x32(t_o + D / 2 + c, b);
+        tmem_ld_wait();
+        if (row_ok) {
+          float fa[32], fb[32];
+#pragma unroll
+          for (int g = 0; g < 8; ++g) {
+            const float4 cv = tr[c / 4 + g], sv = tr[D / 8 + c / 4 + g];
+            const float cs[4] = {cv.x, cv.y, cv.z, cv.w}, sn[4] = {sv.x, sv.y, sv.z, sv.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float u = __uint_as_float(a[g * 4 + e]), w = __uint_as_float(b[g * 4 + e]);
+              fa[g * 4 + e] = u * cs[e] + w * sn[e];
+              fb[g * 4 + e] = w * cs[e] - u * sn[e];
+            }
+          }
+          store32(c, fa);
+          store32(c + D / 2, fb);
+        }
+      }
+    } else {
+#pragma unroll 1
+      for (int c = 0; c < D; c += 32) {
+        uint32_t v[32];
+        tmem_ld_32x32(t_o + c, v);
+        tmem_ld_wait();
+        if (row_ok) {
+          float f[32];
+#pragma unroll
+          for (int e = 0; e < 32; ++e) f[e] = __uint_as_float(v[e]);
+          store32(c, f);
         }
       }
     }
@@ -401,19 +473,19 @@ static int get_kv_slab_tmap(const void* base, int64_t num_pages, int Hkv, int D,
   return 0;
 }
 
-template <int D, int KV, bool CAP = false>
+template <int D, int KV, bool CAP = false, bool BIAS = false>
 static int launch_prefill_tc(const CUtensorMap& tk, const CUtensorMap& tv, const TcAttnParams& p, int num_seqs,
                              int max_q_len, cudaStream_t st) {
   using SM = TcSmem<D, KV>;
   static PerDeviceOnce configured;
   if (configured.need()) {
-    CUDA_CHECK_RET(cudaFuncSetAttribute(attn_prefill_tc_kernel<D, KV, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    CUDA_CHECK_RET(cudaFuncSetAttribute(attn_prefill_tc_kernel<D, KV, CAP, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                         SM::kBytes));
     configured.done();
   }
   const int toks_per_tile = kTcRows / p.GP;
   dim3 grid((max_q_len + toks_per_tile - 1) / toks_per_tile, num_seqs, p.Hkv * (p.G / p.GP));
-  attn_prefill_tc_kernel<D, KV, CAP><<<grid, kTcThreads, SM::kBytes, st>>>(tk, tv, p);
+  attn_prefill_tc_kernel<D, KV, CAP, BIAS><<<grid, kTcThreads, SM::kBytes, st>>>(tk, tv, p);
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
 }
@@ -429,10 +501,11 @@ static int attn_prefill_tc_impl(const void* q, int64_t q_ts, void* out, const vo
                                 int64_t num_pages, const void* block_table, const void* seq_lens,
                                 const void* q_start, int num_seqs, int seq_offset, int max_q_len,
                                 int max_blocks, int Hq, int Hkv, int D, int page_size, float scale, int kv_tile,
-                                const void* sink, float softcap, void* stream) {
+                                const void* sink, float softcap, void* stream, int window = 0, int64_t out_ts = 0,
+                                const AttnExtras& ex = AttnExtras()) {
   if (num_seqs <= 0 || max_q_len <= 0) return 0;
   if ((D != 64 && D != 128) || (kv_tile != 64 && kv_tile != 128) || page_size < 8 || kv_tile % page_size != 0 ||
-      Hq % Hkv != 0)
+      Hq % Hkv != 0 || (ex.r1 != nullptr && softcap > 0.f))
     return 2;
   CUtensorMap tk, tv;
   if (get_kv_slab_tmap(k_cache, num_pages, Hkv, D, page_size, &tk)) return 1;
@@ -452,6 +525,9 @@ static int attn_prefill_tc_impl(const void* q, int64_t q_ts, void* out, const vo
   p.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
   p.scale_over_cap = softcap > 0.f ? scale / softcap : 0.f;
   p.sink = reinterpret_cast<const float*>(sink);
+  p.out_ts = out_ts > 0 ? out_ts : static_cast<int64_t>(Hq) * D;
+  p.window = window;
+  p.ex = ex;
   // MN-major V operand (see the header comment); overridable for bring-up
   p.v_lbo16 = static_cast<uint32_t>(kv_tile * 128) >> 4;
   p.v_sbo16 = 1024 >> 4;
@@ -464,6 +540,14 @@ static int attn_prefill_tc_impl(const void* q, int64_t q_ts, void* out, const vo
     }
   }
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (ex.r1 != nullptr) {
+    if (D == 128) {
+      return kv_tile == 128 ? launch_prefill_tc<128, 128, false, true>(tk, tv, p, num_seqs, max_q_len, st)
+                            : launch_prefill_tc<128, 64, false, true>(tk, tv, p, num_seqs, max_q_len, st);
+    }
+    return kv_tile == 128 ? launch_prefill_tc<64, 128, false, true>(tk, tv, p, num_seqs, max_q_len, st)
+                          : launch_prefill_tc<64, 64, false, true>(tk, tv, p, num_seqs, max_q_len, st);
+  }
   if (softcap > 0.f) {
     if (D == 128) {
       return kv_tile == 128 ? launch_prefill_tc<128, 128, true>(tk, tv, p, num_seqs, max_q_len, st)
@@ -490,14 +574,17 @@ GLLM_EXPORT int gllm_attn_prefill_tc(const void* q, int64_t q_ts, void* out, con
                               stream);
 }
 
-// the same full-causal attention with a per-head softmax sink (null = none) and a tanh cap on the scaled scores
-// (0 = none); output rows are dense ([tokens, Hq * D])
+// the same causal attention with a per-head softmax sink (null = none) and a tanh cap on the scaled scores
+// (0 = none), a sliding window (0 = none) and the options of AttnExtras; output rows are out_ts elements apart (16-byte
+// aligned), gate rows likewise
 GLLM_EXPORT int gllm_attn_prefill_tc_cap(const void* q, int64_t q_ts, void* out, const void* k_cache,
                                          const void* v_cache, int64_t num_pages, const void* block_table,
                                          const void* seq_lens, const void* q_start, int num_seqs, int seq_offset,
                                          int max_q_len, int max_blocks, int Hq, int Hkv, int D, int page_size,
-                                         float scale, int kv_tile, const void* sink, float softcap, void* stream) {
+                                         float scale, int kv_tile, const void* sink, float softcap, int window,
+                                         int64_t out_ts, const void* r1, const void* r2, const void* gate, int64_t ldg,
+                                         const void* v_turn, void* stream) {
   return attn_prefill_tc_impl(q, q_ts, out, k_cache, v_cache, num_pages, block_table, seq_lens, q_start, num_seqs,
                               seq_offset, max_q_len, max_blocks, Hq, Hkv, D, page_size, scale, kv_tile, sink, softcap,
-                              stream);
+                              stream, window, out_ts, make_extras(r1, r2, gate, ldg, v_turn));
 }

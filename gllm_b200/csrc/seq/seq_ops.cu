@@ -33,19 +33,20 @@ __global__ void embed_scale_kernel(const int* __restrict__ ids, const T* __restr
 // x += rms(y) * w_post * post_scale ; x += add ; out = rms(x) * w_pre   (each part optional; post_scale: an fp32
 // layer scale). With emit_plain and no w_pre, out = x rounded to T (sublayers that read the stream un-normed).
 // w_off is added to both norm weights in fp32 (1 for weights stored around zero); out_mul multiplies the normed
-// output (a logit scale applied to the final norm's result, before it is rounded).
+// output (a logit scale applied to the final norm's result, before it is rounded). y_mul multiplies the branch (a
+// residual multiplier); without w_post the branch is added as it is: x += y_mul * y.
 template <typename T>
 __global__ void __launch_bounds__(256) resid_norm_kernel(float* __restrict__ x, const T* __restrict__ y, long ldy,
                                                          const T* __restrict__ w_post,
                                                          const float* __restrict__ post_scale,
                                                          const float* __restrict__ add, const T* __restrict__ w_pre,
                                                          T* __restrict__ out, int width, float eps, int emit_plain,
-                                                         float w_off, float out_mul) {
+                                                         float w_off, float out_mul, float y_mul) {
   __shared__ float scratch[8];
   const int t = blockIdx.x;
   float* xr = x + (size_t)t * width;
-  float r_post = 0.f;
-  if (y != nullptr) {
+  float r_post = 1.f;
+  if (y != nullptr && w_post != nullptr) {
     const T* yr = y + (size_t)t * ldy;
     float ss = 0.f;
     for (int i = threadIdx.x; i < width; i += 256) { float v = to_f(yr[i]); ss += v * v; }
@@ -57,7 +58,9 @@ __global__ void __launch_bounds__(256) resid_norm_kernel(float* __restrict__ x, 
   for (int i = threadIdx.x; i < width; i += 256) {
     float v = xr[i];
     if (y != nullptr) {
-      float br = to_f(y[(size_t)t * ldy + i]) * r_post * (to_f(w_post[i]) + w_off);
+      float br = to_f(y[(size_t)t * ldy + i]);
+      if (w_post != nullptr) br *= r_post * (to_f(w_post[i]) + w_off);
+      br *= y_mul;
       if (post_scale != nullptr) br *= post_scale[i];
       v += br;
     }
@@ -110,13 +113,16 @@ __global__ void qk_norm_kv_write_kernel(const T* __restrict__ qk, long ldqk, int
 // slab widths); the result is multiplied by out_scale and written with row stride ldo. One warp per (token, head);
 // 4 consecutive tokens of one head per block (their key ranges overlap, so K/V rows are shared through L1).
 // Scores: one key per lane; P.V: value entries across lanes. softcap > 0: a scaled score s becomes
-// softcap * tanh(s / softcap) before the softmax.
+// softcap * tanh(s / softcap) before the softmax. r1, r2 (per head, both or none): r1 ln(1 + r2 (i - j)) is taken off the
+// score of key j. v_turn [ntok, Dv] (cos | sin of the query's position per pair): the values are rotated, the result
+// is turned back, entry m with m + Dv / 2. gate (row stride ldg): the result is multiplied by sigmoid(gate).
 template <typename T, int MAXR>
 __global__ void __launch_bounds__(128) window_attn_kernel(
     const T* __restrict__ q, const T* __restrict__ kc, const T* __restrict__ vc, const int* __restrict__ block_table,
     int bt_stride, const int* __restrict__ qsl, const int* __restrict__ positions, int ntok, int nseq, float scale,
     int H, int G, int D, int Dv, int window, int chunk, const float* __restrict__ sink, T* __restrict__ out, long ldo,
-    float out_scale, int ps, int slab, int slab_v, float softcap) {
+    float out_scale, int ps, int slab, int slab_v, float softcap, const float* __restrict__ r1,
+    const float* __restrict__ r2, const T* __restrict__ gate, long ldg, const float* __restrict__ v_turn) {
   __shared__ float qs[4][256];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + warp, h = blockIdx.y;
@@ -155,6 +161,7 @@ __global__ void __launch_bounds__(128) window_attn_kernel(
       }
       sc = dot * scale;
       if (softcap > 0.f) sc = softcap * tanhf(sc / softcap);
+      if (r1 != nullptr) sc -= r1[h] * log1pf(r2[h] * (float)(i - j));
     }
     const float m_new = fmaxf(m, warp_max(sc));
     const float alpha = expf(m - m_new);          // m == -inf only before the first key: exp(-inf) == 0
@@ -176,10 +183,26 @@ __global__ void __launch_bounds__(128) window_attn_kernel(
   }
   T* orow = out + (size_t)t * ldo + (size_t)h * Dv;
   const float inv = out_scale / l;
+  const int half = Dv / 2;
+  const float* turn = v_turn != nullptr ? v_turn + (size_t)t * Dv : nullptr;
+  if (turn != nullptr) {             // the pairs of a head meet through the warp's (now unused) query row
+    __syncwarp();
+#pragma unroll
+    for (int r = 0; r < MAXR; ++r)
+      if (lane + 32 * r < Dv) qs[warp][lane + 32 * r] = acc[r];
+    __syncwarp();
+  }
 #pragma unroll
   for (int r = 0; r < MAXR; ++r) {
     const int d = lane + 32 * r;
-    if (d < Dv) orow[d] = from_f<T>(acc[r] * inv);
+    if (d >= Dv) continue;
+    float v = acc[r];
+    if (turn != nullptr)
+      v = d < half ? v * turn[d] + qs[warp][d + half] * turn[half + d]
+                   : v * turn[d - half] - qs[warp][d - half] * turn[d];
+    v *= inv;
+    if (gate != nullptr) v /= 1.0f + expf(-to_f(gate[(size_t)t * ldg + (size_t)h * Dv + d]));
+    orow[d] = from_f<T>(v);
   }
 }
 
@@ -213,6 +236,76 @@ __global__ void conv_silu_kernel(const T* __restrict__ xz, long ldxz, int C, con
     acc = fmaf(w[(size_t)c * taps + j], v, acc);
   }
   out[(size_t)t * C + c] = from_f<T>(act == 0 ? acc / (1.0f + expf(-acc)) : acc);
+}
+
+// The same convolution for bf16 rows whose channels come in aligned groups of 8: a thread owns 8 channels (16-byte loads
+// and stores, weights in registers) and walks `rows` consecutive batch rows with the last TAPS - 1 inputs in
+// registers, so every input row is read once per block instead of TAPS times. The next row's load is in flight while
+// the current one is computed.
+template <int TAPS>
+__global__ void __launch_bounds__(128) conv_silu_vec_kernel(
+    const __nv_bfloat16* __restrict__ xz, long ldxz, int C, const float* __restrict__ w, const float* __restrict__ b,
+    const __nv_bfloat16* __restrict__ state, const int* __restrict__ rec_slots, const int* __restrict__ seq_lens,
+    const int* __restrict__ qsl, int nseq, int ntok, int rows, __nv_bfloat16* __restrict__ out, int act,
+    const float* __restrict__ in_bias) {
+  const int c = (blockIdx.y * 128 + threadIdx.x) * 8;
+  if (c >= C) return;
+  const int t0 = blockIdx.x * rows, t1 = min(t0 + rows, ntok);
+  float wr[8][TAPS], br[8], ib[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    br[e] = b[c + e];
+    ib[e] = in_bias != nullptr ? in_bias[c + e] : 0.f;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wr[e][j] = w[(size_t)(c + e) * TAPS + j];
+  }
+  auto unpack = [](const uint4 v, float (&f)[8]) {
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 p = __bfloat1622float2(h[e]);
+      f[2 * e] = p.x;
+      f[2 * e + 1] = p.y;
+    }
+  };
+  float win[TAPS][8];                            // win[0 .. TAPS-2]: inputs before the row; win[TAPS-1]: the row's own
+  int s = find_seq(qsl, nseq, t0), q0 = 0, q1 = -1;
+  uint4 cur = *reinterpret_cast<const uint4*>(xz + (size_t)t0 * ldxz + c);
+  for (int t = t0; t < t1; ++t) {
+    const uint4 nxt = t + 1 < t1 ? *reinterpret_cast<const uint4*>(xz + (size_t)(t + 1) * ldxz + c) : cur;
+    if (t >= q1) {                               // first row of the block or of a sequence: gather its past
+      while (s + 1 < nseq && qsl[s + 1] <= t) ++s;
+      q0 = qsl[s];
+      q1 = qsl[s + 1];
+      const int li = t - q0, pos0 = seq_lens[s] - (q1 - q0);
+      const bool carried = state != nullptr && pos0 > 0;
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) {
+        const int src = li - (TAPS - 1) + j;
+        const bool own = src >= 0, have = own || (carried && pos0 + src >= 0);
+        float f[8];
+        if (own) unpack(*reinterpret_cast<const uint4*>(xz + (size_t)(q0 + src) * ldxz + c), f);
+        else if (have)
+          unpack(*reinterpret_cast<const uint4*>(state + ((size_t)rec_slots[s] * (TAPS - 1) + TAPS - 1 + src) * C + c), f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) win[j][e] = have ? f[e] + ib[e] : 0.f;
+      }
+    }
+    unpack(cur, win[TAPS - 1]);
+    __nv_bfloat16 o[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      win[TAPS - 1][e] += ib[e];
+      float acc = br[e];
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) acc = fmaf(wr[e][j], win[j][e], acc);
+      o[e] = __float2bfloat16_rn(act == 0 ? acc / (1.0f + expf(-acc)) : acc);
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS; ++j) win[j][e] = win[j + 1][e];
+    }
+    *reinterpret_cast<uint4*>(out + (size_t)t * C + c) = *reinterpret_cast<const uint4*>(o);
+    cur = nxt;
+  }
 }
 
 // after the convolution: state <- the last taps - 1 inputs of the sequence (shifting in what the chunk brought)
@@ -383,11 +476,13 @@ template <typename T>
 int attn_dispatch(dim3 grid, cudaStream_t st, const void* q, const void* kc, const void* vc, const int* bt,
                   int bt_stride, const int* qsl, const int* pos, int ntok, int nseq, float scale, int H, int G, int D,
                   int Dv, int window, int chunk, const float* sink, void* out, long ldo, float out_scale, int ps,
-                  int slab, int slab_v, float softcap) {
+                  int slab, int slab_v, float softcap, const float* r1, const float* r2, const void* gate, long ldg,
+                  const float* v_turn) {
 #define GLLM_ATTN(R)                                                                                              \
   window_attn_kernel<T, R><<<grid, 128, 0, st>>>((const T*)q, (const T*)kc, (const T*)vc, bt, bt_stride, qsl, pos, \
                                                  ntok, nseq, scale, H, G, D, Dv, window, chunk, sink, (T*)out, ldo, \
-                                                 out_scale, ps, slab, slab_v, softcap)
+                                                 out_scale, ps, slab, slab_v, softcap, r1, r2, (const T*)gate, ldg, \
+                                                 v_turn)
   if (D > 256) return 2;
   if (Dv <= 32) GLLM_ATTN(1);
   else if (Dv <= 64) GLLM_ATTN(2);
@@ -418,18 +513,19 @@ GLLM_EXPORT int gllm_seq_embed_scale(const void* ids, const void* table, void* o
 
 GLLM_EXPORT int gllm_seq_resid_norm(void* x, const void* y, long ldy, const void* w_post, const void* post_scale,
                                     const void* add, const void* w_pre, void* out, int ntok, int width, float eps,
-                                    int emit_plain, int is_f32, float w_off, float out_mul, void* stream) {
+                                    int emit_plain, int is_f32, float w_off, float out_mul, float y_mul,
+                                    void* stream) {
   if (ntok <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
   GLLM_BY_DTYPE(is_f32,
                 (resid_norm_kernel<__nv_bfloat16><<<ntok, 256, 0, st>>>(
                     (float*)x, (const __nv_bfloat16*)y, ldy, (const __nv_bfloat16*)w_post, (const float*)post_scale,
                     (const float*)add, (const __nv_bfloat16*)w_pre, (__nv_bfloat16*)out, width, eps, emit_plain,
-                    w_off, out_mul)),
+                    w_off, out_mul, y_mul)),
                 (resid_norm_kernel<float><<<ntok, 256, 0, st>>>((float*)x, (const float*)y, ldy, (const float*)w_post,
                                                                 (const float*)post_scale, (const float*)add,
                                                                 (const float*)w_pre, (float*)out, width, eps,
-                                                                emit_plain, w_off, out_mul)));
+                                                                emit_plain, w_off, out_mul, y_mul)));
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
 }
@@ -455,19 +551,23 @@ GLLM_EXPORT int gllm_seq_window_attention(const void* q, const void* kc, const v
                                           int bt_stride, const void* qsl, const void* positions, int ntok, int nseq,
                                           float scale, int H, int G, int D, int Dv, int window, int chunk,
                                           const void* sink, void* out, long ldo, float out_scale, int ps, int slab,
-                                          int slab_v, int is_f32, float softcap, void* stream) {
+                                          int slab_v, int is_f32, float softcap, const void* r1, const void* r2,
+                                          const void* gate, long ldg, const void* v_turn, void* stream) {
   if (ntok <= 0) return 0;
+  if (v_turn != nullptr && Dv % 2 != 0) return 2;
   cudaStream_t st = (cudaStream_t)stream;
   dim3 grid((ntok + 3) / 4, H);
   int rc;
   if (is_f32)
     rc = attn_dispatch<float>(grid, st, q, kc, vc, (const int*)block_table, bt_stride, (const int*)qsl,
                               (const int*)positions, ntok, nseq, scale, H, G, D, Dv, window, chunk, (const float*)sink,
-                              out, ldo, out_scale, ps, slab, slab_v, softcap);
+                              out, ldo, out_scale, ps, slab, slab_v, softcap, (const float*)r1, (const float*)r2, gate,
+                              ldg, (const float*)v_turn);
   else
     rc = attn_dispatch<__nv_bfloat16>(grid, st, q, kc, vc, (const int*)block_table, bt_stride, (const int*)qsl,
                                       (const int*)positions, ntok, nseq, scale, H, G, D, Dv, window, chunk,
-                                      (const float*)sink, out, ldo, out_scale, ps, slab, slab_v, softcap);
+                                      (const float*)sink, out, ldo, out_scale, ps, slab, slab_v, softcap,
+                                      (const float*)r1, (const float*)r2, gate, ldg, (const float*)v_turn);
   if (rc) return rc;
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
@@ -488,6 +588,21 @@ GLLM_EXPORT int gllm_seq_conv_silu(const void* xz, long ldxz, int ntok, int nseq
                                                              (const int*)rec_slots, (const int*)seq_lens,
                                                              (const int*)qsl);
   } else {
+    const bool vec = C % 8 == 0 && ldxz % 8 == 0 && ((uintptr_t)xz & 15) == 0 && taps >= 1 && taps <= 4 &&
+                     ((uintptr_t)state & 15) == 0 && ((uintptr_t)out & 15) == 0;
+    const int rows = ntok >= 2048 ? 16 : (ntok >= 512 ? 4 : 1);
+    dim3 vgrid((ntok + rows - 1) / rows, (C / 8 + 127) / 128);
+#define GLLM_CONV_VEC(TAPS)                                                                                        \
+  conv_silu_vec_kernel<TAPS><<<vgrid, 128, 0, st>>>(                                                               \
+      (const __nv_bfloat16*)xz, ldxz, C, (const float*)w, (const float*)b, (const __nv_bfloat16*)state,            \
+      (const int*)rec_slots, (const int*)seq_lens, (const int*)qsl, nseq, ntok, rows, (__nv_bfloat16*)out, act,    \
+      (const float*)in_bias)
+    if (vec && taps == 1) GLLM_CONV_VEC(1);
+    else if (vec && taps == 2) GLLM_CONV_VEC(2);
+    else if (vec && taps == 3) GLLM_CONV_VEC(3);
+    else if (vec) GLLM_CONV_VEC(4);
+    else
+#undef GLLM_CONV_VEC
     conv_silu_kernel<__nv_bfloat16><<<grid, 128, 0, st>>>(
         (const __nv_bfloat16*)xz, ldxz, C, (const float*)w, (const float*)b, taps, (const __nv_bfloat16*)state,
         (const int*)rec_slots, (const int*)seq_lens, (const int*)qsl, nseq, (__nv_bfloat16*)out, act,

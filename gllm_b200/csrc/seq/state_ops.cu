@@ -47,19 +47,27 @@ __global__ void __launch_bounds__(256) postnorm_kernel(float* __restrict__ x, co
 // pos * base^(-2i/rot). The token's cos / sin row is formed once per block, the angle in fp64 (no table, no maximum
 // position), the rotation itself in fp32. `freqs` (fp64, one per pair) replaces the powers of the base (scaled
 // frequencies); cos and sin are multiplied by `mag`. With G == 0 a row holds queries only (the keys and values are
-// another layer's) and no cache is touched.
+// another layer's) and no cache is touched. `unit`: q / k are divided by their root mean square without a weight.
+// `angles` [ntok, rot] (cos | sin, fp32): the row's table as formed once per step, used instead of positions and
+// frequencies; `v_angles` [ntok, Dv]: the values turn too, entry m with m + Dv / 2, and are cached so.
 template <typename T>
 __global__ void __launch_bounds__(256) qk_norm_rope_kv_write_kernel(
     const T* __restrict__ qkv, long ld, int H, int G, int D, int Dv, const T* __restrict__ qn,
     const T* __restrict__ kn, float eps, const int* __restrict__ positions, int rot, double log2_base,
     T* __restrict__ q_out, T* __restrict__ kc, T* __restrict__ vc, const int* __restrict__ slots, int ps, int slab,
-    int slab_v, const double* __restrict__ freqs, float mag) {
+    int slab_v, const double* __restrict__ freqs, float mag, int unit, const float* __restrict__ angles,
+    const float* __restrict__ v_angles) {
   extern __shared__ float cs_tab[];      // [rot / 2] cos, then [rot / 2] sin
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x;
   const int half = rot / 2;
   const double pos = (double)positions[t];
   for (int i = threadIdx.x; i < half; i += 256) {
+    if (angles != nullptr) {
+      cs_tab[i] = angles[(size_t)t * rot + i] * mag;
+      cs_tab[half + i] = angles[(size_t)t * rot + half + i] * mag;
+      continue;
+    }
     double sn, cs;
     sincos(pos * (freqs != nullptr ? freqs[i] : exp2(-(2.0 * (double)i / (double)rot) * log2_base)), &sn, &cs);
     cs_tab[i] = (float)(cs * (double)mag);
@@ -72,7 +80,15 @@ __global__ void __launch_bounds__(256) qk_norm_rope_kv_write_kernel(
       if (slot < 0) continue;
       const int g = head - H - G;
       const T* src = qkv + (size_t)t * ld + (size_t)(H + G) * D + (size_t)g * Dv;
-      for (int d = lane; d < Dv; d += 32) vc[cache_index(slot, g, d, G, Dv, ps, slab_v)] = src[d];
+      const float* va = v_angles != nullptr ? v_angles + (size_t)t * Dv : nullptr;
+      const int vh = Dv / 2;
+      for (int d = lane; d < Dv; d += 32) {
+        T o = src[d];
+        if (va != nullptr)
+          o = from_f<T>(d < vh ? to_f(o) * va[d] - to_f(src[d + vh]) * va[vh + d]
+                               : to_f(o) * va[d - vh] + to_f(src[d - vh]) * va[d]);
+        vc[cache_index(slot, g, d, G, Dv, ps, slab_v)] = o;
+      }
       continue;
     }
     if (head >= H && slot < 0) continue;
@@ -81,7 +97,7 @@ __global__ void __launch_bounds__(256) qk_norm_rope_kv_write_kernel(
     for (int d = lane; d < D; d += 32) { const float v = to_f(src[d]); ss += v * v; }
     ss = warp_sum(ss);
     const T* w = head < H ? qn : kn;
-    const float r = w != nullptr ? 1.0f / sqrtf(ss / (float)D + eps) : 1.0f;
+    const float r = w != nullptr || unit ? 1.0f / sqrtf(ss / (float)D + eps) : 1.0f;
     for (int d = lane; d < D; d += 32) {
       float v = to_f(src[d]) * r * (w != nullptr ? to_f(w[d]) : 1.0f);
       if (d < rot) {
@@ -103,7 +119,8 @@ __global__ void __launch_bounds__(256) qk_norm_rope_kv_write_kernel(
 // registers per thread, twice the warps in flight). q / k rows and the per-token g, beta of TCH tokens are staged
 // in shared memory by the whole block (SiLU, unit length and the q scale applied there). With KD the decay is one
 // value per key channel, gk[t, h * D + d] in fp32 (`key_decay_kernel`), acting on row d; it is staged beside the key as
-// (k, decay) pairs, so the update still costs two shared loads per state entry.
+// (k, decay) pairs, so the update still costs two shared loads per state entry. `step`: the softplus that forms the
+// decay is also the write strength (u = softplus(a + dt_bias) v); dskip (per head): o += dskip v.
 template <typename T, int NS, int PARTS, bool KD>
 __global__ void __launch_bounds__(32 * PARTS) linear_state_kernel(
     const T* __restrict__ q, long ldq, const T* __restrict__ k, long ldk, const T* __restrict__ v, long ldv,
@@ -111,7 +128,7 @@ __global__ void __launch_bounds__(32 * PARTS) linear_state_kernel(
     const float* __restrict__ dt_bias, const float* __restrict__ decay, float* __restrict__ state,
     const int* __restrict__ rec_slots, const int* __restrict__ seq_lens, const int* __restrict__ qsl, int H, int G,
     int D, int V, int silu_in, int unit_qk, float q_scale, int delta, float* __restrict__ out,
-    const float* __restrict__ gk, long ldgk) {
+    const float* __restrict__ gk, long ldgk, int step, const float* __restrict__ dskip) {
   constexpr int TCH = 8;               // tokens staged per round (16 measured 2.4x slower: registers)
   constexpr int ROWS = KD ? 3 : 2;
   extern __shared__ float sm[];
@@ -162,7 +179,9 @@ __global__ void __launch_bounds__(32 * PARTS) linear_state_kernel(
         g = decay[h];
       } else {
         const float z = to_f(a[(size_t)(t0 + threadIdx.x) * lda + h]) + dt_bias[h];
-        g = expf(neg_a[h] * (z > 20.0f ? z : log1pf(expf(z))));
+        const float sp = z > 20.0f ? z : log1pf(expf(z));
+        g = expf(neg_a[h] * sp);
+        if (step) b = sp;
       }
       if (delta) b = sigmoid_f(to_f(beta[(size_t)(t0 + threadIdx.x) * ldb + h]));
       sg[threadIdx.x * 2] = g;
@@ -209,6 +228,8 @@ __global__ void __launch_bounds__(32 * PARTS) linear_state_kernel(
 #pragma unroll
           for (int o = 1; o < PARTS; o <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
           u = b * (u - g * dot);
+        } else if (step) {
+          u *= b;
         }
         float o = 0.f;
 #pragma unroll
@@ -226,6 +247,7 @@ __global__ void __launch_bounds__(32 * PARTS) linear_state_kernel(
         }
 #pragma unroll
         for (int sh = 1; sh < PARTS; sh <<= 1) o += __shfl_xor_sync(0xffffffffu, o, sh);
+        if (dskip != nullptr) o = fmaf(dskip[h], vv[kk], o);
         if (active && part == 0) out[(size_t)(t0 + kk) * H * V + (size_t)h * V + vcol] = o;
       }
     }
@@ -263,11 +285,12 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ o, int n, cons
 }
 
 template <typename T>
-__global__ void silu_mul_kernel(const T* __restrict__ gu, long ld, int F, T* __restrict__ out, size_t total) {
+__global__ void silu_mul_kernel(const T* __restrict__ gu, long ld, int F, T* __restrict__ out, long ldo,
+                                size_t total) {
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= total) return;
   const size_t t = i / F, f = i - t * F;
-  out[i] = from_f<T>(silu_f(to_f(gu[t * ld + f])) * to_f(gu[t * ld + F + f]));
+  out[t * ldo + f] = from_f<T>(silu_f(to_f(gu[t * ld + f])) * to_f(gu[t * ld + F + f]));
 }
 
 // Router logits for small batches: one warp per (token, expert), lanes over the width in a fixed order, fp32 result.
@@ -553,11 +576,12 @@ int state_dispatch(dim3 grid, size_t smem, cudaStream_t st, const void* q, long 
                    const void* v, long ldv, const void* beta, long ldb, const void* a, long lda, const float* neg_a,
                    const float* dt_bias, const float* decay, float* state, const int* rec_slots, const int* seq_lens,
                    const int* qsl, int H, int G, int D, int V, int silu_in, int unit_qk, float q_scale, int delta,
-                   float* out, int parts, const float* zk, long ldz) {
+                   float* out, int parts, const float* zk, long ldz, int step, const float* dskip) {
 #define GLLM_STATE_KD(NS, PARTS, KD)                                                                                \
   linear_state_kernel<T, NS, PARTS, KD><<<grid, 32 * PARTS, smem, st>>>(                                            \
       (const T*)q, ldq, (const T*)k, ldk, (const T*)v, ldv, (const T*)beta, ldb, (const T*)a, lda, neg_a, dt_bias,  \
-      decay, state, rec_slots, seq_lens, qsl, H, G, D, V, silu_in, unit_qk, q_scale, delta, out, zk, ldz)
+      decay, state, rec_slots, seq_lens, qsl, H, G, D, V, silu_in, unit_qk, q_scale, delta, out, zk, ldz, \
+      step, dskip)
 #define GLLM_STATE(NS, PARTS)                                               \
   do {                                                                      \
     if (zk != nullptr) GLLM_STATE_KD(NS, PARTS, true);                      \
@@ -597,7 +621,8 @@ GLLM_EXPORT int gllm_seq_qk_norm_rope_kv_write(const void* qkv, long ld, int nto
                                                const void* qn, const void* kn, float eps, const void* positions,
                                                int rot, double log2_base, void* q_out, void* kc, void* vc,
                                                const void* slots, int ps, int slab, int slab_v, int is_f32,
-                                               const void* freqs, float mag, void* stream) {
+                                               const void* freqs, float mag, int unit, const void* angles,
+                                               const void* v_angles, void* stream) {
   if (ntok <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
   dim3 grid(ntok);
@@ -606,11 +631,13 @@ GLLM_EXPORT int gllm_seq_qk_norm_rope_kv_write(const void* qkv, long ld, int nto
                 (qk_norm_rope_kv_write_kernel<bf16_t><<<grid, 256, smem, st>>>(
                     (const bf16_t*)qkv, ld, H, G, D, Dv, (const bf16_t*)qn, (const bf16_t*)kn, eps,
                     (const int*)positions, rot, log2_base, (bf16_t*)q_out, (bf16_t*)kc, (bf16_t*)vc,
-                    (const int*)slots, ps, slab, slab_v, (const double*)freqs, mag)),
+                    (const int*)slots, ps, slab, slab_v, (const double*)freqs, mag, unit, (const float*)angles,
+                    (const float*)v_angles)),
                 (qk_norm_rope_kv_write_kernel<float><<<grid, 256, smem, st>>>(
                     (const float*)qkv, ld, H, G, D, Dv, (const float*)qn, (const float*)kn, eps,
                     (const int*)positions, rot, log2_base, (float*)q_out, (float*)kc, (float*)vc, (const int*)slots,
-                    ps, slab, slab_v, (const double*)freqs, mag)));
+                    ps, slab, slab_v, (const double*)freqs, mag, unit, (const float*)angles,
+                    (const float*)v_angles)));
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
 }
@@ -620,8 +647,10 @@ GLLM_EXPORT int gllm_seq_linear_state(const void* q, long ldq, const void* k, lo
                                       const void* dt_bias, const void* decay, void* state, const void* rec_slots,
                                       const void* seq_lens, const void* qsl, int nseq, int H, int G, int D, int V,
                                       int silu_in, int unit_qk, float q_scale, int delta, void* out, int is_f32,
-                                      int parts, const void* gk, long ldgk, void* stream) {
+                                      int parts, const void* gk, long ldgk, int step, const void* dskip,
+                                      void* stream) {
   if (nseq <= 0) return 0;
+  if (step && (delta || a == nullptr)) return 2;                       // the step is the decay's own softplus
   if (gk != nullptr && (delta || G != H)) return 2;                    // key-channel decay: plain update, own keys
   cudaStream_t st = (cudaStream_t)stream;
   dim3 grid(nseq, H, (V + 31) / 32);
@@ -632,12 +661,12 @@ GLLM_EXPORT int gllm_seq_linear_state(const void* q, long ldq, const void* k, lo
     rc = state_dispatch<float>(grid, smem, st, q, ldq, k, ldk, v, ldv, beta, ldb, a, lda, (const float*)neg_a,
                                (const float*)dt_bias, (const float*)decay, (float*)state, (const int*)rec_slots,
                                (const int*)seq_lens, (const int*)qsl, H, G, D, V, silu_in, unit_qk, q_scale, delta,
-                               (float*)out, parts, (const float*)gk, ldgk);
+                               (float*)out, parts, (const float*)gk, ldgk, step, (const float*)dskip);
   else
     rc = state_dispatch<bf16_t>(grid, smem, st, q, ldq, k, ldk, v, ldv, beta, ldb, a, lda, (const float*)neg_a,
                                 (const float*)dt_bias, (const float*)decay, (float*)state, (const int*)rec_slots,
                                 (const int*)seq_lens, (const int*)qsl, H, G, D, V, silu_in, unit_qk, q_scale, delta,
-                                (float*)out, parts, (const float*)gk, ldgk);
+                                (float*)out, parts, (const float*)gk, ldgk, step, (const float*)dskip);
   if (rc) return rc;
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
@@ -662,14 +691,15 @@ GLLM_EXPORT int gllm_seq_gated_group_norm(const void* o, int n, const void* gate
   return 0;
 }
 
-GLLM_EXPORT int gllm_seq_silu_mul(const void* gu, long ld, int ntok, int F, void* out, int is_f32, void* stream) {
+GLLM_EXPORT int gllm_seq_silu_mul(const void* gu, long ld, int ntok, int F, void* out, long ldo, int is_f32,
+                                  void* stream) {
   if (ntok <= 0 || F <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
   const size_t total = (size_t)ntok * F;
   const unsigned blocks = (unsigned)((total + 255) / 256);
   GLLM_BY_DTYPE(is_f32,
-                (silu_mul_kernel<bf16_t><<<blocks, 256, 0, st>>>((const bf16_t*)gu, ld, F, (bf16_t*)out, total)),
-                (silu_mul_kernel<float><<<blocks, 256, 0, st>>>((const float*)gu, ld, F, (float*)out, total)));
+                (silu_mul_kernel<bf16_t><<<blocks, 256, 0, st>>>((const bf16_t*)gu, ld, F, (bf16_t*)out, ldo, total)),
+                (silu_mul_kernel<float><<<blocks, 256, 0, st>>>((const float*)gu, ld, F, (float*)out, ldo, total)));
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
 }

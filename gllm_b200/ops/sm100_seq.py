@@ -26,18 +26,19 @@ def _L():
         P, I, G, F = c_void_p, c_int, c_long, c_float
         sigs = {
             "gllm_seq_embed_scale": [P, P, P, I, I, I, F, I, P],
-            "gllm_seq_resid_norm": [P, P, G, P, P, P, P, P, I, I, F, I, I, F, F, P],
+            "gllm_seq_resid_norm": [P, P, G, P, P, P, P, P, I, I, F, I, I, F, F, F, P],
             "gllm_seq_qk_norm_kv_write": [P, G, I, I, I, I, P, P, F, P, P, P, P, I, I, I, P],
-            "gllm_seq_window_attention": [P, P, P, P, I, P, P, I, I, F, I, I, I, I, I, I, P, P, G, F, I, I, I, I, F, P],
+            "gllm_seq_window_attention": [P, P, P, P, I, P, P, I, I, F, I, I, I, I, I, I, P, P, G, F, I, I, I, I, F, P, P, P, G,
+                                          P, P],
             "gllm_seq_postnorm": [P, P, G, P, P, I, I, F, F, I, P],
             "gllm_seq_qk_norm_rope_kv_write": [P, G, I, I, I, I, I, P, P, F, P, I, ctypes.c_double, P, P, P, P, I, I, I,
-                                               I, P, F, P],
+                                               I, P, F, I, P, P, P],
             "gllm_seq_linear_state": [P, G, P, G, P, G, P, G, P, G, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, P,
-                                      I, I, P, G, P],
+                                      I, I, P, G, I, P, P],
             "gllm_seq_key_decay": [P, G, P, F, P, I, I, I, P],
             "gllm_seq_gemm_mma_f32out": [P, G, G, P, G, G, P, G, G, I, I, I, I, P],
             "gllm_seq_gated_group_norm": [P, I, P, G, P, I, I, F, I, F, P, G, I, I, P],
-            "gllm_seq_silu_mul": [P, G, I, I, P, I, P],
+            "gllm_seq_silu_mul": [P, G, I, I, P, G, I, P],
             "gllm_seq_router_select": [P, I, I, I, P, P, P],
             "gllm_seq_router_logits": [P, G, P, I, I, I, P, I, P],
             "gllm_seq_router_logits_mma": [P, G, P, I, I, I, P, P],
@@ -50,9 +51,11 @@ def _L():
             "gllm_seq_gemm_simt": [P, G, P, G, P, G, I, I, I, I, P, P],
             "gllm_attn_decode_win": [P, G, P, P, P, G, P, P, I, I, I, I, I, I, I, F, I, P, P],
             "gllm_attn_prefill_win": [P, G, P, P, P, G, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
-            "gllm_attn_prefill_tc_cap": [P, G, P, P, P, G, P, P, P, I, I, I, I, I, I, I, I, F, I, P, F, P],
-            "gllm_attn_decode_mask": [P, G, P, G, P, P, G, P, P, I, I, I, I, I, I, I, F, I, I, P, F, F, P],
-            "gllm_attn_prefill_mask": [P, G, P, G, P, P, G, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, F, F, P],
+            "gllm_attn_prefill_tc_cap": [P, G, P, P, P, G, P, P, P, I, I, I, I, I, I, I, I, F, I, P, F, I, G, P, P, P, G, P,
+                                         P],
+            "gllm_attn_decode_mask": [P, G, P, G, P, P, G, P, P, I, I, I, I, I, I, I, F, I, I, P, F, F, P, P, P, G, P, P],
+            "gllm_attn_prefill_mask": [P, G, P, G, P, P, G, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, F, F, P, P, P, G, P,
+                                       P],
         }
         for name, args in sigs.items():
             fn = getattr(L, name)
@@ -102,7 +105,7 @@ def embedding_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float) -> to
 
 
 def resid_norm(x, y, w_post, add, w_pre, eps, out_dtype, emit_plain=False, post_scale=None, w_offset=0.0,
-               out_mul=1.0):
+               out_mul=1.0, y_mul=1.0):
     assert x.dtype == torch.float32 and x.is_contiguous()
     t, width = x.shape
     plain = bool(emit_plain) and w_pre is None
@@ -112,11 +115,11 @@ def resid_norm(x, y, w_post, add, w_pre, eps, out_dtype, emit_plain=False, post_
         ret_x = False
     out = torch.empty(t, width, dtype=out_dtype, device=x.device) if (w_pre is not None or plain) else None
     assert post_scale is None or (post_scale.dtype == torch.float32 and post_scale.is_contiguous())
-    ref_t = w_pre if w_pre is not None else (w_post if w_post is not None else None)
+    ref_t = w_pre if w_pre is not None else (w_post if w_post is not None else y)
     is32 = 1 if (ref_t is not None and ref_t.dtype == torch.float32) or (ref_t is None and out_dtype == torch.float32) \
         else 0
     if y is not None:
-        assert y.stride(1) == 1 and y.dtype == w_post.dtype
+        assert y.stride(1) == 1 and (ref_t is None or y.dtype == ref_t.dtype)
     if add is not None:
         assert add.dtype == torch.float32 and add.is_contiguous()
     if y is None and add is None and w_pre is None and not plain:
@@ -144,12 +147,16 @@ def qk_norm_kv_write(qk, num_heads, num_kv_heads, dim, q_norm_w, k_norm_w, eps, 
 def window_attention(q, k_cache, v_cache, block_table, seq_lens, query_start_loc, positions, scale, num_q_heads,
                      head_dim, window, sink, num_decode_seqs: int = 0, max_q_len: Optional[int] = None,
                      simt: bool = False, chunk: Optional[int] = None, v_dim: Optional[int] = None,
-                     out_scale: float = 1.0, out: Optional[torch.Tensor] = None, softcap: float = 0.0):
+                     out_scale: float = 1.0, out: Optional[torch.Tensor] = None, softcap: float = 0.0, dist_bias=None,
+                     gate: Optional[torch.Tensor] = None, v_turn: Optional[torch.Tensor] = None,
+                     tc: Optional[bool] = None):
     """Masked paged attention: sliding window (None / 0 = full causal) and / or chunk mask, optional per-head softmax
     sink, values `v_dim` wide, result times `out_scale` into `out` (any row stride). bf16 with v_dim == head_dim
     in 64 / 128 / 256 and pages of 8..64 tokens runs on the tensor-core paged-attention kernels
     (csrc/attn/paged_attention.cu: the first `num_decode_seqs` sequences, one token each, on the decode kernel, the
-    rest on the prefill kernel); everything else (fp32, other head sizes or page sizes) on the plain kernel."""
+    rest on the tcgen05 prefill kernel for head sizes 64 / 128 without a chunk mask, else on the mma.sync prefill
+    kernel; `tc=False` keeps the latter); everything else (fp32, other head sizes or page sizes) on the plain kernel.
+    `dist_bias`, `gate`, `v_turn`: see `ops.ref.window_attention`."""
     t = q.shape[0]
     v_dim = head_dim if v_dim is None else v_dim
     if out is None:
@@ -160,6 +167,18 @@ def window_attention(q, k_cache, v_cache, block_table, seq_lens, query_start_loc
     nseq = seq_lens.shape[0]
     # the tensor-core kernels store 8-byte vectors: rows and head offsets of `out` must keep that alignment
     tc_ok = v_dim == head_dim and out.stride(0) % 4 == 0 and out.data_ptr() % 8 == 0
+    r1, r2 = dist_bias if dist_bias is not None else (None, None)
+    assert r1 is None or (r1.dtype == torch.float32 == r2.dtype and r1.is_contiguous() and r2.is_contiguous())
+    assert v_turn is None or (v_turn.dtype == torch.float32 and v_turn.is_contiguous() and
+                              v_turn.shape == (t, v_dim))
+    ldg = 0
+    if gate is not None:
+        assert gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (t, num_q_heads * v_dim)
+        ldg = gate.stride(0)
+        tc_ok = tc_ok and ldg % 4 == 0 and gate.data_ptr() % 8 == 0
+    vec16 = out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 and \
+        (gate is None or (ldg % 8 == 0 and gate.data_ptr() % 16 == 0))
+    extras = (_p(r1), _p(r2), _p(gate), ldg, _p(v_turn))
     if not simt and tc_ok and q.dtype == torch.bfloat16 and head_dim in (64, 128, 256) and slab == 64 and ps >= 8 and \
             64 % ps == 0 and max_q_len is not None:
         L, st = _L(), stream_ptr()
@@ -168,17 +187,17 @@ def window_attention(q, k_cache, v_cache, block_table, seq_lens, query_start_loc
             check(L.gllm_attn_decode_mask(_p(q), q.stride(0), _p(out), out.stride(0), _p(k_cache), _p(v_cache), pages,
                                           _p(block_table), _p(seq_lens), num_decode_seqs, 0, block_table.stride(0),
                                           num_q_heads, hkv, head_dim, ps, float(scale), int(window or 0),
-                                          int(chunk or 0), _p(sink), float(out_scale), float(softcap), st),
+                                          int(chunk or 0), _p(sink), float(out_scale), float(softcap), *extras, st),
                   "attn_decode_mask")
             sm100._count()
         rest = nseq > num_decode_seqs
-        if rest and not window and not chunk and sm100.ATTN_TC and out_scale == 1.0 and \
-                out.stride(0) == num_q_heads * head_dim and head_dim in (64, 128) and sm100.ATTN_TC_KV % ps == 0:
-            # full causal (cap and sink only): the tcgen05 prefill kernel
+        if rest and not chunk and sm100.ATTN_TC and out_scale == 1.0 and vec16 and tc is not False and \
+                head_dim in (64, 128) and sm100.ATTN_TC_KV % ps == 0:
             rc = L.gllm_attn_prefill_tc_cap(_p(q), q.stride(0), _p(out), _p(k_cache), _p(v_cache), pages,
                                             _p(block_table), _p(seq_lens), _p(query_start_loc), nseq - num_decode_seqs,
                                             num_decode_seqs, max_q_len, block_table.stride(0), num_q_heads, hkv,
-                                            head_dim, ps, float(scale), sm100.ATTN_TC_KV, _p(sink), float(softcap), st)
+                                            head_dim, ps, float(scale), sm100.ATTN_TC_KV, _p(sink), float(softcap),
+                                            int(window or 0), out.stride(0), *extras, st)
             if rc != 2:                     # 2 = shape outside that kernel's envelope -> the mma.sync kernel
                 check(rc, "attn_prefill_tc_cap")
                 sm100._count()
@@ -188,14 +207,14 @@ def window_attention(q, k_cache, v_cache, block_table, seq_lens, query_start_loc
                                            _p(block_table), _p(seq_lens), _p(query_start_loc), nseq - num_decode_seqs,
                                            num_decode_seqs, max_q_len, block_table.stride(0), num_q_heads, hkv,
                                            head_dim, ps, float(scale), int(window or 0), int(chunk or 0), _p(sink),
-                                           float(out_scale), float(softcap), st), "attn_prefill_mask")
+                                           float(out_scale), float(softcap), *extras, st), "attn_prefill_mask")
             sm100._count()
         return out
     check(_L().gllm_seq_window_attention(_p(q), _p(k_cache), _p(v_cache), _p(block_table), block_table.stride(0),
                                          _p(query_start_loc), _p(positions), t, seq_lens.shape[0], float(scale),
                                          num_q_heads, k_cache.shape[1], head_dim, v_dim, int(window or 0),
                                          int(chunk or 0), _p(sink), _p(out), out.stride(0), float(out_scale), ps, slab,
-                                         v_cache.shape[4], _f32(q), float(softcap), stream_ptr()),
+                                         v_cache.shape[4], _f32(q), float(softcap), *extras, stream_ptr()),
           "seq_window_attention")
     sm100._count()
     return out
@@ -248,33 +267,41 @@ def postnorm(x, y, alpha, w, eps, out_dtype):
 
 
 def qk_norm_rope_kv_write(qkv, num_heads, num_kv_heads, dim, v_dim, q_norm_w, k_norm_w, eps, positions, rot_dims,
-                          rot_base, k_cache, v_cache, slots, freqs=None, mag=1.0):
+                          rot_base, k_cache, v_cache, slots, freqs=None, mag=1.0, unit_norm=False, angles=None,
+                          v_angles=None):
     import math
     t = qkv.shape[0]
     assert qkv.stride(1) == 1 and k_cache.dtype == qkv.dtype and positions.dim() == 1
     assert freqs is None or (freqs.dtype == torch.float64 and freqs.is_contiguous() and
                              freqs.shape[0] == rot_dims // 2)
+    assert angles is None or (angles.dtype == torch.float32 and angles.is_contiguous() and
+                              angles.shape == (t, rot_dims))
+    assert v_angles is None or (v_angles.dtype == torch.float32 and v_angles.is_contiguous() and
+                                v_angles.shape == (t, v_dim))
     q = torch.empty(t, num_heads * dim, dtype=qkv.dtype, device=qkv.device)
     ps = k_cache.shape[3]
     check(_L().gllm_seq_qk_norm_rope_kv_write(_p(qkv), qkv.stride(0), t, num_heads, num_kv_heads, dim, v_dim,
                                               _p(q_norm_w), _p(k_norm_w), float(eps), _p(positions), int(rot_dims),
                                               math.log2(rot_base) if rot_dims > 0 else 0.0, _p(q), _p(k_cache),
                                               _p(v_cache), _p(slots), ps, k_cache.shape[4], v_cache.shape[4],
-                                              _f32(qkv), _p(freqs), float(mag), stream_ptr()),
+                                              _f32(qkv), _p(freqs), float(mag), int(unit_norm), _p(angles),
+                                              _p(v_angles), stream_ptr()),
           "seq_qk_norm_rope_kv_write")
     sm100._count()
     return q
 
 
 def linear_state_scan(q, k, v, beta, a, neg_a, dt_bias, decay, state, rec_slots, seq_lens, query_start_loc, heads,
-                      qk_heads, dim, v_dim, silu_in, unit_qk, q_scale, delta, zk=None, zk_bias=None, inv_tau=1.0):
+                      qk_heads, dim, v_dim, silu_in, unit_qk, q_scale, delta, zk=None, zk_bias=None, inv_tau=1.0,
+                      step=False, d_skip=None, out=None):
+    """`step`: the softplus behind the decay is also the write strength; `d_skip` [heads] fp32: o += d_skip v."""
     t = q.shape[0]
     for x in (q, k, v, beta, a, zk):
         assert x is None or (x.stride(1) == 1 and x.dtype == q.dtype)
     assert state is None or (state.dtype == torch.float32 and state.is_contiguous())
     assert (decay is not None) + (a is not None) + (zk is not None) == 1 and (not delta or beta is not None)
     assert zk_bias is None or (zk_bias.dtype == torch.float32 and zk_bias.is_contiguous())
-    out = torch.empty(t, heads * v_dim, dtype=torch.float32, device=q.device)
+    out = torch.empty(t, heads * v_dim, dtype=torch.float32, device=q.device) if out is None else out
     ld = lambda x: x.stride(0) if x is not None else 0   # noqa: E731
     gk = None
     if zk is not None:
@@ -293,7 +320,7 @@ def linear_state_scan(q, k, v, beta, a, neg_a, dt_bias, decay, state, rec_slots,
                                      _p(a), ld(a), _p(neg_a), _p(dt_bias), _p(decay), _p(state), _p(rec_slots),
                                      _p(seq_lens), _p(query_start_loc), seq_lens.shape[0], heads, qk_heads, dim, v_dim,
                                      int(silu_in), int(unit_qk), float(q_scale), int(delta), _p(out), _f32(q),
-                                     parts, _p(gk), ld(gk), stream_ptr()), "seq_linear_state")
+                                     parts, _p(gk), ld(gk), int(step), _p(d_skip), stream_ptr()), "seq_linear_state")
     sm100._count()
     return out
 
@@ -311,11 +338,12 @@ def gated_group_norm(o, gate, w, group, eps, act, out_scale=1.0, out=None, out_d
     return out
 
 
-def silu_mul(gu):
+def silu_mul(gu, out=None):
     t, f = gu.shape[0], gu.shape[1] // 2
-    assert gu.stride(1) == 1
-    out = torch.empty(t, f, dtype=gu.dtype, device=gu.device)
-    check(_L().gllm_seq_silu_mul(_p(gu), gu.stride(0), t, f, _p(out), _f32(gu), stream_ptr()), "seq_silu_mul")
+    out = torch.empty(t, f, dtype=gu.dtype, device=gu.device) if out is None else out
+    assert gu.stride(1) == 1 and out.stride(1) == 1 and out.shape == (t, f) and out.dtype == gu.dtype
+    check(_L().gllm_seq_silu_mul(_p(gu), gu.stride(0), t, f, _p(out), out.stride(0), _f32(gu), stream_ptr()),
+          "seq_silu_mul")
     sm100._count()
     return out
 
