@@ -126,7 +126,7 @@ def resid_norm(x, y, w_post, add, w_pre, eps, out_dtype, emit_plain=False, post_
         return x if ret_x else None
     check(_L().gllm_seq_resid_norm(_p(x), _p(y), y.stride(0) if y is not None else 0, _p(w_post), _p(post_scale),
                                    _p(add), _p(w_pre), _p(out), t, width, float(eps), int(plain), is32, float(w_offset),
-                                   float(out_mul), stream_ptr()),
+                                   float(out_mul), float(y_mul), stream_ptr()),
           "seq_resid_norm")
     sm100._count()
     return x if ret_x else out
