@@ -77,6 +77,106 @@ __global__ void __launch_bounds__(256) resid_norm_kernel(float* __restrict__ x, 
 }
 
 
+// The same update for bf16 rows of 8-wide aligned pieces: a thread keeps its up to MAXP pieces of the row in registers,
+// so the fp32 stream is read once and written once with 16-byte accesses.
+template <int MAXP>
+__global__ void __launch_bounds__(256) resid_norm_vec_kernel(
+    float* __restrict__ x, const __nv_bfloat16* __restrict__ y, long ldy, const __nv_bfloat16* __restrict__ w_post,
+    const float* __restrict__ post_scale, const float* __restrict__ add, const __nv_bfloat16* __restrict__ w_pre,
+    __nv_bfloat16* __restrict__ out, int width, float eps, int emit_plain, float w_off, float out_mul, float y_mul) {
+  __shared__ float scratch[8];
+  const size_t row = (size_t)blockIdx.x * width;
+  auto load8 = [](const __nv_bfloat16* ptr, float (&f)[8]) {
+    const uint4 v = *reinterpret_cast<const uint4*>(ptr);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 p = __bfloat1622float2(h[e]);
+      f[2 * e] = p.x;
+      f[2 * e + 1] = p.y;
+    }
+  };
+  auto load8f = [](const float* ptr, float (&f)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(ptr), b = *reinterpret_cast<const float4*>(ptr + 4);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+    f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+  };
+  auto store8 = [](__nv_bfloat16* ptr, const float (&f)[8]) {
+    __align__(16) __nv_bfloat162 h[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) h[e] = __floats2bfloat162_rn(f[2 * e], f[2 * e + 1]);
+    *reinterpret_cast<uint4*>(ptr) = *reinterpret_cast<const uint4*>(h);
+  };
+  float v[MAXP][8], b[MAXP][8];
+  float r_post = 1.f, ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < MAXP; ++k) {
+    const int i = (threadIdx.x + k * 256) * 8;
+    if (i < width) {
+      load8f(x + row + i, v[k]);
+      if (y != nullptr) {
+        load8(y + (size_t)blockIdx.x * ldy + i, b[k]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss += b[k][e] * b[k][e];
+      }
+    }
+  }
+  if (y != nullptr && w_post != nullptr) {
+    ss = block_sum<256>(ss, scratch);
+    r_post = 1.0f / sqrtf(ss / (float)width + eps);
+  }
+  const bool plain = w_pre == nullptr && emit_plain && out != nullptr;
+  float ss2 = 0.f;
+#pragma unroll
+  for (int k = 0; k < MAXP; ++k) {
+    const int i = (threadIdx.x + k * 256) * 8;
+    if (i < width) {
+      if (y != nullptr) {
+        float w[8];
+        if (w_post != nullptr) {
+          load8(w_post + i, w);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) b[k][e] *= r_post * (w[e] + w_off);
+        }
+        if (post_scale != nullptr) {
+          load8f(post_scale + i, w);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) b[k][e] *= w[e];
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[k][e] = fmaf(b[k][e], y_mul, v[k][e]);
+      }
+      if (add != nullptr) {
+        float a[8];
+        load8f(add + row + i, a);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[k][e] += a[e];
+      }
+      if (y != nullptr || add != nullptr) {
+        *reinterpret_cast<float4*>(x + row + i) = make_float4(v[k][0], v[k][1], v[k][2], v[k][3]);
+        *reinterpret_cast<float4*>(x + row + i + 4) = make_float4(v[k][4], v[k][5], v[k][6], v[k][7]);
+      }
+      if (plain) store8(out + row + i, v[k]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss2 += v[k][e] * v[k][e];
+    }
+  }
+  if (w_pre == nullptr) return;
+  ss2 = block_sum<256>(ss2, scratch);
+  const float r = 1.0f / sqrtf(ss2 / (float)width + eps);
+#pragma unroll
+  for (int k = 0; k < MAXP; ++k) {
+    const int i = (threadIdx.x + k * 256) * 8;
+    if (i < width) {
+      float w[8];
+      load8(w_pre + i, w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) w[e] = v[k][e] * r * (w[e] + w_off) * out_mul;
+      store8(out + row + i, w);
+    }
+  }
+}
+
 // one warp per (token, head): heads [0, H) are queries, [H, H + G) keys
 template <typename T>
 __global__ void qk_norm_kv_write_kernel(const T* __restrict__ qk, long ldqk, int ntok, int H, int G, int D,
@@ -241,24 +341,25 @@ __global__ void conv_silu_kernel(const T* __restrict__ xz, long ldxz, int C, con
 // The same convolution for bf16 rows whose channels come in aligned groups of 8: a thread owns 8 channels (16-byte loads
 // and stores, weights in registers) and walks `rows` consecutive batch rows with the last TAPS - 1 inputs in
 // registers, so every input row is read once per block instead of TAPS times. The next row's load is in flight while
-// the current one is computed.
+// the current one is computed. Sequences of one token also update their carried inputs here (longer ones: the kernel
+// below, after every block has read them).
 template <int TAPS>
 __global__ void __launch_bounds__(128) conv_silu_vec_kernel(
     const __nv_bfloat16* __restrict__ xz, long ldxz, int C, const float* __restrict__ w, const float* __restrict__ b,
-    const __nv_bfloat16* __restrict__ state, const int* __restrict__ rec_slots, const int* __restrict__ seq_lens,
+    __nv_bfloat16* __restrict__ state, const int* __restrict__ rec_slots, const int* __restrict__ seq_lens,
     const int* __restrict__ qsl, int nseq, int ntok, int rows, __nv_bfloat16* __restrict__ out, int act,
     const float* __restrict__ in_bias) {
   const int c = (blockIdx.y * 128 + threadIdx.x) * 8;
   if (c >= C) return;
   const int t0 = blockIdx.x * rows, t1 = min(t0 + rows, ntok);
-  float wr[8][TAPS], br[8], ib[8];
+  __align__(16) float wr[8 * TAPS], br[8], ib[8];              // weight of channel e, tap j: wr[e * TAPS + j]
 #pragma unroll
-  for (int e = 0; e < 8; ++e) {
-    br[e] = b[c + e];
-    ib[e] = in_bias != nullptr ? in_bias[c + e] : 0.f;
+  for (int e = 0; e < 8 * TAPS; e += 4)
+    *reinterpret_cast<float4*>(wr + e) = *reinterpret_cast<const float4*>(w + (size_t)c * TAPS + e);
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) wr[e][j] = w[(size_t)(c + e) * TAPS + j];
-  }
+  for (int e = 0; e < 8; e += 4) *reinterpret_cast<float4*>(br + e) = *reinterpret_cast<const float4*>(b + c + e);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) ib[e] = in_bias != nullptr ? in_bias[c + e] : 0.f;
   auto unpack = [](const uint4 v, float (&f)[8]) {
     const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
 #pragma unroll
@@ -292,32 +393,43 @@ __global__ void __launch_bounds__(128) conv_silu_vec_kernel(
       }
     }
     unpack(cur, win[TAPS - 1]);
-    __nv_bfloat16 o[8];
+    __align__(16) __nv_bfloat16 o[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) {
       win[TAPS - 1][e] += ib[e];
       float acc = br[e];
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) acc = fmaf(wr[e][j], win[j][e], acc);
-      o[e] = __float2bfloat16_rn(act == 0 ? acc / (1.0f + expf(-acc)) : acc);
+      for (int j = 0; j < TAPS; ++j) acc = fmaf(wr[e * TAPS + j], win[j][e], acc);
+      o[e] = __float2bfloat16_rn(act == 0 ? acc * __fdividef(1.0f, 1.0f + __expf(-acc)) : acc);
 #pragma unroll
       for (int j = 0; j + 1 < TAPS; ++j) win[j][e] = win[j + 1][e];
     }
     *reinterpret_cast<uint4*>(out + (size_t)t * C + c) = *reinterpret_cast<const uint4*>(o);
+    if (TAPS > 1 && state != nullptr && q1 - q0 == 1) {
+      // a single token's sequence: nobody else reads its slot, so the carried inputs move up here
+      __nv_bfloat16* st = state + (size_t)rec_slots[s] * (TAPS - 1) * C + c;
+      const bool carried = seq_lens[s] > 1;
+#pragma unroll
+      for (int j = 0; j + 1 < TAPS - 1; ++j)
+        *reinterpret_cast<uint4*>(st + (size_t)j * C) =
+            carried ? *reinterpret_cast<const uint4*>(st + (size_t)(j + 1) * C) : make_uint4(0u, 0u, 0u, 0u);
+      *reinterpret_cast<uint4*>(st + (size_t)(TAPS - 2) * C) = cur;
+    }
     cur = nxt;
   }
 }
 
-// after the convolution: state <- the last taps - 1 inputs of the sequence (shifting in what the chunk brought)
+// after the convolution: state <- the last taps - 1 inputs of the sequence (shifting in what the chunk brought);
+// sequences shorter than `min_len` tokens are skipped (they have been updated already)
 template <typename T>
 __global__ void conv_state_update_kernel(const T* __restrict__ xz, long ldxz, int C, int taps, T* __restrict__ state,
                                          const int* __restrict__ rec_slots, const int* __restrict__ seq_lens,
-                                         const int* __restrict__ qsl) {
+                                         const int* __restrict__ qsl, int min_len) {
   const int s = blockIdx.x;
   const int c = blockIdx.y * blockDim.x + threadIdx.x;
   if (c >= C || taps < 2) return;
   const int q0 = qsl[s], n = qsl[s + 1] - q0;
-  if (n <= 0) return;
+  if (n < min_len) return;
   const bool carried = (seq_lens[s] - n) > 0;
   T* st = state + (size_t)rec_slots[s] * (taps - 1) * C;
   for (int k = 0; k < taps - 1; ++k) {           // ascending k reads index k + n > k: never an overwritten entry
@@ -517,6 +629,21 @@ GLLM_EXPORT int gllm_seq_resid_norm(void* x, const void* y, long ldy, const void
                                     void* stream) {
   if (ntok <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
+  const uintptr_t al = (uintptr_t)x | (uintptr_t)y | (uintptr_t)w_post | (uintptr_t)post_scale | (uintptr_t)add |
+                       (uintptr_t)w_pre | (uintptr_t)out;
+  if (!is_f32 && width % 8 == 0 && width >= 512 && width <= 8192 && ldy % 8 == 0 && (al & 15) == 0) {
+#define GLLM_RESID(MP)                                                                                              \
+  resid_norm_vec_kernel<MP><<<ntok, 256, 0, st>>>((float*)x, (const __nv_bfloat16*)y, ldy,                          \
+                                                  (const __nv_bfloat16*)w_post, (const float*)post_scale,           \
+                                                  (const float*)add, (const __nv_bfloat16*)w_pre,                   \
+                                                  (__nv_bfloat16*)out, width, eps, emit_plain, w_off, out_mul, y_mul)
+    if (width <= 2048) GLLM_RESID(1);
+    else if (width <= 4096) GLLM_RESID(2);
+    else GLLM_RESID(4);
+#undef GLLM_RESID
+    CUDA_CHECK_RET(cudaGetLastError());
+    return 0;
+  }
   GLLM_BY_DTYPE(is_f32,
                 (resid_norm_kernel<__nv_bfloat16><<<ntok, 256, 0, st>>>(
                     (float*)x, (const __nv_bfloat16*)y, ldy, (const __nv_bfloat16*)w_post, (const float*)post_scale,
@@ -575,7 +702,8 @@ GLLM_EXPORT int gllm_seq_window_attention(const void* q, const void* kc, const v
 
 GLLM_EXPORT int gllm_seq_conv_silu(const void* xz, long ldxz, int ntok, int nseq, int C, const void* w, const void* b,
                                    int taps, void* state, const void* rec_slots, const void* seq_lens, const void* qsl,
-                                   void* out, int is_f32, int act, const void* in_bias, void* stream) {
+                                   void* out, int is_f32, int act, const void* in_bias, int max_q_len,
+                                   void* stream) {
   if (ntok <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
   dim3 grid(ntok, (C + 127) / 128), sgrid(nseq, (C + 127) / 128);
@@ -586,15 +714,16 @@ GLLM_EXPORT int gllm_seq_conv_silu(const void* xz, long ldxz, int ntok, int nseq
     if (state != nullptr && taps > 1)
       conv_state_update_kernel<float><<<sgrid, 128, 0, st>>>((const float*)xz, ldxz, C, taps, (float*)state,
                                                              (const int*)rec_slots, (const int*)seq_lens,
-                                                             (const int*)qsl);
+                                                             (const int*)qsl, 1);
   } else {
     const bool vec = C % 8 == 0 && ldxz % 8 == 0 && ((uintptr_t)xz & 15) == 0 && taps >= 1 && taps <= 4 &&
-                     ((uintptr_t)state & 15) == 0 && ((uintptr_t)out & 15) == 0;
+                     ((uintptr_t)state & 15) == 0 && ((uintptr_t)out & 15) == 0 && ((uintptr_t)w & 15) == 0 &&
+                     ((uintptr_t)b & 15) == 0;
     const int rows = ntok >= 2048 ? 16 : (ntok >= 512 ? 4 : 1);
     dim3 vgrid((ntok + rows - 1) / rows, (C / 8 + 127) / 128);
 #define GLLM_CONV_VEC(TAPS)                                                                                        \
   conv_silu_vec_kernel<TAPS><<<vgrid, 128, 0, st>>>(                                                               \
-      (const __nv_bfloat16*)xz, ldxz, C, (const float*)w, (const float*)b, (const __nv_bfloat16*)state,            \
+      (const __nv_bfloat16*)xz, ldxz, C, (const float*)w, (const float*)b, (__nv_bfloat16*)state,                  \
       (const int*)rec_slots, (const int*)seq_lens, (const int*)qsl, nseq, ntok, rows, (__nv_bfloat16*)out, act,    \
       (const float*)in_bias)
     if (vec && taps == 1) GLLM_CONV_VEC(1);
@@ -607,10 +736,10 @@ GLLM_EXPORT int gllm_seq_conv_silu(const void* xz, long ldxz, int ntok, int nseq
         (const __nv_bfloat16*)xz, ldxz, C, (const float*)w, (const float*)b, taps, (const __nv_bfloat16*)state,
         (const int*)rec_slots, (const int*)seq_lens, (const int*)qsl, nseq, (__nv_bfloat16*)out, act,
         (const float*)in_bias);
-    if (state != nullptr && taps > 1)
+    if (state != nullptr && taps > 1 && !(vec && max_q_len == 1))
       conv_state_update_kernel<__nv_bfloat16><<<sgrid, 128, 0, st>>>(
           (const __nv_bfloat16*)xz, ldxz, C, taps, (__nv_bfloat16*)state, (const int*)rec_slots, (const int*)seq_lens,
-          (const int*)qsl);
+          (const int*)qsl, vec ? 2 : 1);
   }
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;

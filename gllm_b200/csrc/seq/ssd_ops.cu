@@ -208,8 +208,9 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(
 // so a chunk is four small matrix products on the tensor cores and only S is carried from chunk to chunk (in fp32
 // accumulators). C, B and x are exact bf16; the fp32 operands (S, the weighted scores, the weighted x) are split into
 // a bf16 head and a bf16 remainder and multiplied twice, which keeps 16 significant bits of each.
-// One block per (sequence, head, VT value columns), four warps, warp w = tokens 16 w .. 16 w + 15 of the chunk in the
-// output products and a share of the state rows (WM warps) and value columns (4 / WM) in the state update.
+// One block per (sequence, head, VT value columns), NW = 4 or 8 warps: warp w works on tokens 16 (w % 4) .. + 15 of the
+// chunk and on one of NW / 4 shares of the value columns in the output products, and on a share of the state rows (WM
+// warps) and value columns (NW / WM) in the state update.
 constexpr int kQ = 64;
 
 __device__ __forceinline__ uint32_t s_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -249,8 +250,8 @@ struct SsdSmem {
   static constexpr int kBytes = kElems * 2 + 5 * kQ * 4;
 };
 
-template <int NP, int VT>
-__global__ void __launch_bounds__(128) ssd_chunk_kernel(
+template <int NP, int VT, int NW>
+__global__ void __launch_bounds__(32 * NW, NW == 8 ? 2 : 1) ssd_chunk_kernel(
     const bf16_t* __restrict__ x, long ldx, const bf16_t* __restrict__ b, long ldb, const bf16_t* __restrict__ c,
     long ldc, const bf16_t* __restrict__ dt, long lddt, const float* __restrict__ neg_a,
     const float* __restrict__ dt_bias, const float* __restrict__ d_skip, float* __restrict__ state,
@@ -258,9 +259,10 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(
     int N, int V, float* __restrict__ out) {
   using SM = SsdSmem<NP, VT>;
   constexpr int LN = SM::LN, LV = SM::LV;
-  constexpr int MT = NP / 16, WM = MT < 4 ? MT : 4, WN = 4 / WM;
+  constexpr int NT = 32 * NW, CS = NW / 4, VC = VT / 8 / CS;   // column shares; 8-wide column tiles of a warp's share
+  constexpr int MT = NP / 16, WM = MT < NW ? MT : NW, WN = NW / WM;
   constexpr int MI = MT / WM, NI = VT / 8 / WN;   // state tiles (16 x 8) of a warp
-  static_assert(NI % 2 == 0, "column tiles come in pairs");
+  static_assert(NI % 2 == 0 && VC % 2 == 0, "column tiles come in pairs");
   extern __shared__ __align__(16) uint8_t smem_raw[];
   bf16_t* sm = reinterpret_cast<bf16_t*>(smem_raw);
   bf16_t *sB = sm + SM::B, *sC = sm + SM::C, *sX = sm + SM::X, *sSh = sm + SM::SH, *sSl = sm + SM::SL,
@@ -275,6 +277,7 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(
   const int g4 = lane >> 2, t4 = lane & 3, lq = lane >> 3, lr = lane & 7;
   const int grp = h / (H / G);
   const int wm = warp % WM, wn = warp / WM;
+  const int tw = warp & 3, cb = (warp >> 2) * VC;    // output products: token group, first column tile
   const bool carried = state != nullptr && seq_lens[s] > q1 - q0;
   float* st = state != nullptr ? state + ((size_t)rec_slots[s] * H + h) * (size_t)N * V : nullptr;
   const float na = neg_a[h], db = dt_bias[h], ds = d_skip[h];
@@ -296,14 +299,14 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(
   for (int t0 = q0; t0 < q1; t0 += kQ) {
     const int nt = min(kQ, q1 - t0);
     __syncthreads();                              // the previous chunk's tiles are consumed
-    for (int i = threadIdx.x; i < kQ * (NP / 8); i += 128) {
+    for (int i = threadIdx.x; i < kQ * (NP / 8); i += NT) {
       const int r = i / (NP / 8), e = (i % (NP / 8)) * 8;
       const bool ok = r < nt && e < N;
       const size_t row = t0 + (ok ? r : 0);
       cp16(sB + r * LN + e, bp + row * ldb + (ok ? e : 0), ok);
       cp16(sC + r * LN + e, cp + row * ldc + (ok ? e : 0), ok);
     }
-    for (int i = threadIdx.x; i < kQ * (VT / 8); i += 128) {
+    for (int i = threadIdx.x; i < kQ * (VT / 8); i += NT) {
       const int r = i / (VT / 8), e = (i % (VT / 8)) * 8;
       const bool ok = r < nt && v0 + e < V;
       const size_t row = t0 + (ok ? r : 0);
@@ -349,7 +352,7 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(
     }
     asm volatile("cp.async.wait_group 0;");
     __syncthreads();
-    for (int i = threadIdx.x; i < kQ * (VT / 2); i += 128) {
+    for (int i = threadIdx.x; i < kQ * (VT / 2); i += NT) {
       const int r = i / (VT / 2), e = (i % (VT / 2)) * 2;
       const float2 xv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sX + r * LV + e));
       const float w = sWt[r];
@@ -359,19 +362,19 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(
       *reinterpret_cast<uint32_t*>(sWl + r * LV + e) = lo;
     }
     // ---- C . S (entering state) and C . B^T for this warp's 16 tokens
-    float acc[VT / 8][4], G2[8][4];
+    float acc[VC][4], G2[8][4];
 #pragma unroll
-    for (int i = 0; i < VT / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    for (int i = 0; i < VC; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 #pragma unroll
     for (int i = 0; i < 8; ++i) G2[i][0] = G2[i][1] = G2[i][2] = G2[i][3] = 0.f;
 #pragma unroll
     for (int ks = 0; ks < NP / 16; ++ks) {
       uint32_t a[4];
-      ldsm4(s_addr(sC + (warp * 16 + (lq & 1) * 8 + lr) * LN + ks * 16 + (lq >> 1) * 8), a);
+      ldsm4(s_addr(sC + (tw * 16 + (lq & 1) * 8 + lr) * LN + ks * 16 + (lq >> 1) * 8), a);
 #pragma unroll
-      for (int nv = 0; nv < VT / 8; nv += 2) {
+      for (int nv = 0; nv < VC; nv += 2) {
         uint32_t r[4];
-        const int off = (ks * 16 + (lq & 1) * 8 + lr) * LV + nv * 8 + (lq >> 1) * 8;
+        const int off = (ks * 16 + (lq & 1) * 8 + lr) * LV + (cb + nv) * 8 + (lq >> 1) * 8;
         ldsm4_t(s_addr(sSh + off), r);
         mma16816(acc[nv], a, r[0], r[1]);
         mma16816(acc[nv + 1], a, r[2], r[3]);
@@ -381,7 +384,7 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(
       }
 #pragma unroll
       for (int jt = 0; jt < 8; jt += 2) {
-        if (jt <= 2 * warp) {                     // keys after the warp's last token are not needed
+        if (jt <= 2 * tw) {                     // keys after the warp's last token are not needed
           uint32_t r[4];
           ldsm4(s_addr(sB + (jt * 8 + (lq >> 1) * 8 + lr) * LN + ks * 16 + (lq & 1) * 8), r);
           mma16816(G2[jt], a, r[0], r[1]);
@@ -389,15 +392,15 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(
         }
       }
     }
-    const int ta = warp * 16 + g4, tb = ta + 8;
+    const int ta = tw * 16 + g4, tb = ta + 8;
     const float ea = sEl[ta], eb = sEl[tb];
 #pragma unroll
-    for (int i = 0; i < VT / 8; ++i) { acc[i][0] *= ea; acc[i][1] *= ea; acc[i][2] *= eb; acc[i][3] *= eb; }
+    for (int i = 0; i < VC; ++i) { acc[i][0] *= ea; acc[i][1] *= ea; acc[i][2] *= eb; acc[i][3] *= eb; }
     // ---- weighted scores times x
     const float lha = sLh[ta], lla = sLl[ta], lhb = sLh[tb], llb = sLl[tb];
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk) {
-      if (kk <= warp) {
+      if (kk <= tw) {
         uint32_t ph[4], pl[4];
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
@@ -413,9 +416,9 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(
           split2(p[2], p[3], ph[2 * half + 1], pl[2 * half + 1]);
         }
 #pragma unroll
-        for (int nv = 0; nv < VT / 8; nv += 2) {
+        for (int nv = 0; nv < VC; nv += 2) {
           uint32_t r[4];
-          ldsm4_t(s_addr(sX + (kk * 16 + (lq & 1) * 8 + lr) * LV + nv * 8 + (lq >> 1) * 8), r);
+          ldsm4_t(s_addr(sX + (kk * 16 + (lq & 1) * 8 + lr) * LV + (cb + nv) * 8 + (lq >> 1) * 8), r);
           mma16816(acc[nv], ph, r[0], r[1]);
           mma16816(acc[nv + 1], ph, r[2], r[3]);
           mma16816(acc[nv], pl, r[0], r[1]);
@@ -424,10 +427,10 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(
       }
     }
 #pragma unroll
-    for (int i = 0; i < VT / 8; ++i)
+    for (int i = 0; i < VC; ++i)
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
-        const int tk = r == 0 ? ta : tb, vv = i * 8 + 2 * t4;
+        const int tk = r == 0 ? ta : tb, vv = (cb + i) * 8 + 2 * t4;
         if (tk < nt && v0 + vv < V) {
           const float2 xv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sX + tk * LV + vv));
           *reinterpret_cast<float2*>(out + (size_t)(t0 + tk) * H * V + (size_t)h * V + v0 + vv) =
@@ -478,14 +481,14 @@ __global__ void __launch_bounds__(128) ssd_chunk_kernel(
   }
 }
 
-template <int NP, int VT>
+template <int NP, int VT, int NW>
 int launch_chunk(int nseq, cudaStream_t stm, const void* x, long ldx, const void* b, long ldb, const void* c, long ldc,
                  const void* dt, long lddt, const float* neg_a, const float* dt_bias, const float* d_skip, float* state,
                  const int* rec_slots, const int* seq_lens, const int* qsl, int H, int G, int N, int V, float* out) {
   using SM = SsdSmem<NP, VT>;
-  CUDA_CHECK_RET(cudaFuncSetAttribute(ssd_chunk_kernel<NP, VT>, cudaFuncAttributeMaxDynamicSharedMemorySize, SM::kBytes));
+  CUDA_CHECK_RET(cudaFuncSetAttribute(ssd_chunk_kernel<NP, VT, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, SM::kBytes));
   dim3 grid(H, (V + VT - 1) / VT, nseq);
-  ssd_chunk_kernel<NP, VT><<<grid, 128, SM::kBytes, stm>>>(
+  ssd_chunk_kernel<NP, VT, NW><<<grid, 32 * NW, SM::kBytes, stm>>>(
       (const bf16_t*)x, ldx, (const bf16_t*)b, ldb, (const bf16_t*)c, ldc, (const bf16_t*)dt, lddt, neg_a, dt_bias,
       d_skip, state, rec_slots, seq_lens, qsl, H, G, N, V, out);
   CUDA_CHECK_RET(cudaGetLastError());
@@ -600,13 +603,15 @@ GLLM_EXPORT int gllm_ssd_chunk(const void* x, long ldx, const void* b, long ldb,
       ((uintptr_t)x & 15) != 0 || ((uintptr_t)b & 15) != 0 || ((uintptr_t)c & 15) != 0 || ((uintptr_t)out & 7) != 0)
     return 2;
   cudaStream_t st = (cudaStream_t)stream;
-#define GLLM_CHUNK(NP, VT)                                                                                          \
-  return launch_chunk<NP, VT>(nseq, st, x, ldx, b, ldb, c, ldc, dt, lddt, (const float*)neg_a, (const float*)dt_bias, \
+#define GLLM_CHUNK(NP, VT, NW)                                                                                          \
+  return launch_chunk<NP, VT, NW>(nseq, st, x, ldx, b, ldb, c, ldc, dt, lddt, (const float*)neg_a, (const float*)dt_bias, \
                               (const float*)d_skip, (float*)state, (const int*)rec_slots, (const int*)seq_lens,      \
                               (const int*)qsl, H, G, N, V, (float*)out)
-  if (N <= 32) { if (V <= 32) GLLM_CHUNK(32, 32); else GLLM_CHUNK(32, 64); }
-  if (N <= 64) { if (V <= 32) GLLM_CHUNK(64, 32); else GLLM_CHUNK(64, 64); }
-  if (N <= 128) { if (V <= 32) GLLM_CHUNK(128, 32); else GLLM_CHUNK(128, 64); }
-  GLLM_CHUNK(256, 32);
+  // narrower column blocks where 64-wide ones leave SMs idle (every column is computed alike in both)
+  const bool narrow = V <= 32 || (long)H * nseq * ((V + 63) / 64) <= 148;
+  if (N <= 32) { if (narrow) GLLM_CHUNK(32, 32, 4); else GLLM_CHUNK(32, 64, 8); }
+  if (N <= 64) { if (narrow) GLLM_CHUNK(64, 32, 8); else GLLM_CHUNK(64, 64, 8); }
+  if (N <= 128) { if (narrow) GLLM_CHUNK(128, 32, 8); else GLLM_CHUNK(128, 64, 8); }
+  GLLM_CHUNK(256, 32, 8);
 #undef GLLM_CHUNK
 }

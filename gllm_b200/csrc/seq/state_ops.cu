@@ -112,6 +112,82 @@ __global__ void __launch_bounds__(256) qk_norm_rope_kv_write_kernel(
   }
 }
 
+// The same for bf16 heads whose every entry turns (rot == D) or none does (rot == 0), with the angles given as rows: L
+// lanes per head (D = 8 L; a value head: Dv = 8 L), a lane holding entries 4 l .. 4 l + 3 and their partners D / 2 further,
+// so all traffic is in 8-byte pieces and a rotation stays inside the lane. `lanes` = max(L) over the head kinds.
+__global__ void __launch_bounds__(256) rope_kv_write_vec_kernel(
+    const __nv_bfloat16* __restrict__ qkv, long ld, int H, int G, int D, int Dv, const __nv_bfloat16* __restrict__ qn,
+    const __nv_bfloat16* __restrict__ kn, float eps, __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ kc,
+    __nv_bfloat16* __restrict__ vc, const int* __restrict__ slots, int ps, int slab, int slab_v, float mag, int unit,
+    const float* __restrict__ angles, const float* __restrict__ v_angles, int lanes) {
+  const int t = blockIdx.x;
+  const int l = threadIdx.x % lanes, per = 256 / lanes;
+  const int slot = slots[t];
+  const int total = H + 2 * G, rounds = (total + per - 1) / per;
+  for (int r = 0; r < rounds; ++r) {             // every lane takes every round: the shuffles below need whole warps
+    const int head = r * per + threadIdx.x / lanes;
+    const bool is_v = head >= H + G, on = head < total && (head < H || slot >= 0);
+    const int dim = is_v ? Dv : D, half = dim / 2;
+    const bool mine = on && l * 8 < dim;
+    const __nv_bfloat16* src = qkv + (size_t)t * ld +
+                               (is_v ? (size_t)(H + G) * D + (size_t)(head - H - G) * Dv : (size_t)head * D);
+    float u[4], v[4];
+    float ss = 0.f;
+    if (mine) {
+      const uint2 a = *reinterpret_cast<const uint2*>(src + 4 * l), b = *reinterpret_cast<const uint2*>(src + half + 4 * l);
+      const float2 a0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.x));
+      const float2 a1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.y));
+      const float2 b0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&b.x));
+      const float2 b1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&b.y));
+      u[0] = a0.x; u[1] = a0.y; u[2] = a1.x; u[3] = a1.y;
+      v[0] = b0.x; v[1] = b0.y; v[2] = b1.x; v[3] = b1.y;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) ss += u[e] * u[e] + v[e] * v[e];
+    }
+    for (int o = lanes / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!mine) continue;
+    const __nv_bfloat16* w = head < H ? qn : kn;
+    if (!is_v && (w != nullptr || unit)) {
+      const float rn = 1.0f / sqrtf(ss / (float)D + eps);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        u[e] *= rn * (w != nullptr ? to_f(w[4 * l + e]) : 1.0f);
+        v[e] *= rn * (w != nullptr ? to_f(w[half + 4 * l + e]) : 1.0f);
+      }
+    }
+    const float* ang = is_v ? (v_angles != nullptr ? v_angles + (size_t)t * Dv : nullptr)
+                            : (angles != nullptr ? angles + (size_t)t * D : nullptr);
+    if (ang != nullptr) {
+      const float4 cv = *reinterpret_cast<const float4*>(ang + 4 * l);
+      const float4 sv = *reinterpret_cast<const float4*>(ang + half + 4 * l);
+      const float m = is_v ? 1.0f : mag;
+      const float cs[4] = {cv.x * m, cv.y * m, cv.z * m, cv.w * m}, sn[4] = {sv.x * m, sv.y * m, sv.z * m, sv.w * m};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float p = u[e] * cs[e] - v[e] * sn[e];
+        v[e] = v[e] * cs[e] + u[e] * sn[e];
+        u[e] = p;
+      }
+    }
+    __nv_bfloat162 o0 = __floats2bfloat162_rn(u[0], u[1]), o1 = __floats2bfloat162_rn(u[2], u[3]);
+    __nv_bfloat162 p0 = __floats2bfloat162_rn(v[0], v[1]), p1 = __floats2bfloat162_rn(v[2], v[3]);
+    const uint2 lo = make_uint2(*reinterpret_cast<const uint32_t*>(&o0), *reinterpret_cast<const uint32_t*>(&o1));
+    const uint2 hi = make_uint2(*reinterpret_cast<const uint32_t*>(&p0), *reinterpret_cast<const uint32_t*>(&p1));
+    __nv_bfloat16 *d0, *d1;
+    if (head < H) {
+      d0 = q_out + (size_t)t * H * D + (size_t)head * D + 4 * l;
+      d1 = d0 + half;
+    } else {
+      __nv_bfloat16* base = is_v ? vc : kc;
+      const int g = is_v ? head - H - G : head - H, sl = is_v ? slab_v : slab;
+      d0 = base + cache_index(slot, g, 4 * l, G, dim, ps, sl);
+      d1 = base + cache_index(slot, g, half + 4 * l, G, dim, ps, sl);
+    }
+    *reinterpret_cast<uint2*>(d0) = lo;
+    *reinterpret_cast<uint2*>(d1) = hi;
+  }
+}
+
 // Matrix-state recurrence, one block per (sequence, head, 32 value columns). A value column's D state entries are
 // split over PARTS adjacent lanes (entry d = part + PARTS j), NS per lane in registers; per token
 //     S <- g S;  u = delta ? beta (v - S^T k) : v;  S <- S + k u^T;  o = S^T q
@@ -626,6 +702,21 @@ GLLM_EXPORT int gllm_seq_qk_norm_rope_kv_write(const void* qkv, long ld, int nto
   if (ntok <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
   dim3 grid(ntok);
+  {
+    auto pow2 = [](int v) { return v > 0 && (v & (v - 1)) == 0; };
+    const uintptr_t al = (uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)kc | (uintptr_t)vc;
+    const uintptr_t al16 = (uintptr_t)angles | (uintptr_t)v_angles;
+    if (!is_f32 && G > 0 && (rot == 0 || (rot == D && angles != nullptr)) && D % 8 == 0 && Dv % 8 == 0 && pow2(D / 8) &&
+        pow2(Dv / 8) && D <= 256 && Dv <= 256 && ld % 4 == 0 && (al & 7) == 0 && (al16 & 15) == 0 && slab % 4 == 0 &&
+        slab_v % 4 == 0) {
+      rope_kv_write_vec_kernel<<<grid, 256, 0, st>>>(
+          (const bf16_t*)qkv, ld, H, G, D, Dv, (const bf16_t*)qn, (const bf16_t*)kn, eps, (bf16_t*)q_out, (bf16_t*)kc,
+          (bf16_t*)vc, (const int*)slots, ps, slab, slab_v, mag, unit, rot > 0 ? (const float*)angles : nullptr,
+          (const float*)v_angles, (D > Dv ? D : Dv) / 8);
+      CUDA_CHECK_RET(cudaGetLastError());
+      return 0;
+    }
+  }
   const size_t smem = (size_t)(rot > 0 ? rot : 2) * sizeof(float);
   GLLM_BY_DTYPE(is_f32,
                 (qk_norm_rope_kv_write_kernel<bf16_t><<<grid, 256, smem, st>>>(

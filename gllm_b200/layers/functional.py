@@ -154,8 +154,10 @@ def causal_conv_silu(xz, channels, w, b, conv_state, inp, act="silu", in_bias=No
     """Depthwise causal convolution with carried taps; `act` "silu" | "none"; `in_bias` is added to every input
     that exists (not to the zeros before a sequence's start)."""
     slots = inp.rec_slots if conv_state is not None else None
-    fn = _seq().causal_conv_silu if xz.is_cuda else ref.causal_conv_silu
-    return fn(xz, channels, w, b, conv_state, slots, inp.seq_lens, inp.query_start_loc, act, in_bias)
+    if xz.is_cuda:
+        return _seq().causal_conv_silu(xz, channels, w, b, conv_state, slots, inp.seq_lens, inp.query_start_loc, act,
+                                       in_bias, getattr(inp, "max_q_len", None))
+    return ref.causal_conv_silu(xz, channels, w, b, conv_state, slots, inp.seq_lens, inp.query_start_loc, act, in_bias)
 
 
 def selective_scan(xc, dt_raw, proj, xz, a, d_skip, dt_bias, ssm_state, inp, channels, nstate, dt_rank):

@@ -45,7 +45,7 @@ def _L():
             "gllm_seq_gemm_simt_f32out": [P, G, P, G, P, G, I, I, I, I, P],
             "gllm_seq_routed_experts": [P, G, P, P, P, P, I, I, I, I, P, P, I, I, F, F, I, P],
             "gllm_seq_softcap": [P, G, I, I, F, I, P],
-            "gllm_seq_conv_silu": [P, G, I, I, I, P, P, I, P, P, P, P, P, I, I, P, P],
+            "gllm_seq_conv_silu": [P, G, I, I, I, P, P, I, P, P, P, P, P, I, I, P, I, P],
             "gllm_seq_selective_scan": [P, P, P, G, P, G, P, P, P, P, P, P, P, I, I, I, I, P, I, I, P],
             "gllm_seq_relu2": [P, P, G, I, P],
             "gllm_seq_gemm_simt": [P, G, P, G, P, G, I, I, I, I, P, P],
@@ -220,14 +220,17 @@ def window_attention(q, k_cache, v_cache, block_table, seq_lens, query_start_loc
     return out
 
 
-def causal_conv_silu(xz, channels, w, b, conv_state, rec_slots, seq_lens, query_start_loc, act="silu", in_bias=None):
+def causal_conv_silu(xz, channels, w, b, conv_state, rec_slots, seq_lens, query_start_loc, act="silu", in_bias=None,
+                     max_q_len: Optional[int] = None):
+    """`max_q_len` == 1 tells that every sequence has one token (no separate update of the carried inputs then)."""
     t = xz.shape[0]
     assert xz.stride(1) == 1 and w.dtype == torch.float32 and b.dtype == torch.float32
     assert in_bias is None or (in_bias.dtype == torch.float32 and in_bias.is_contiguous())
     out = torch.empty(t, channels, dtype=xz.dtype, device=xz.device)
     check(_L().gllm_seq_conv_silu(_p(xz), xz.stride(0), t, seq_lens.shape[0], channels, _p(w), _p(b), w.shape[1],
                                   _p(conv_state), _p(rec_slots), _p(seq_lens), _p(query_start_loc), _p(out), _f32(xz),
-                                  0 if act == "silu" else 1, _p(in_bias), stream_ptr()), "seq_conv_silu")
+                                  0 if act == "silu" else 1, _p(in_bias), int(max_q_len or 0), stream_ptr()),
+          "seq_conv_silu")
     sm100._count(2 if conv_state is not None else 1)
     return out
 
