@@ -36,6 +36,7 @@ template <int NT> __device__ __forceinline__ float block_sum(float v, float* scr
 }
 // sequence that owns batch row t: largest s with qsl[s] <= t
 __device__ __forceinline__ int find_seq(const int* __restrict__ qsl, int nseq, int t) {
+  if (t < nseq && qsl[t] <= t && t < qsl[t + 1]) return t;   // single-token sequences lead the batch: row t is theirs
   int lo = 0, hi = nseq - 1;
   while (lo < hi) {
     int mid = (lo + hi + 1) >> 1;

@@ -125,7 +125,7 @@ __global__ void __launch_bounds__(256) gate_then_norm_vec_kernel(
 // accesses. A thread owns 4 value columns and every (256 / (V / 4))-th state row, ROWS rows in flight; partial
 // outputs of the row groups meet in shared memory in a fixed order.
 template <typename T>
-__global__ void __launch_bounds__(256) ssd_step_kernel(
+__global__ void __launch_bounds__(256, 4) ssd_step_kernel(
     const T* __restrict__ x, long ldx, const T* __restrict__ b, long ldb, const T* __restrict__ c, long ldc,
     const T* __restrict__ dt, long lddt, const float* __restrict__ neg_a, const float* __restrict__ dt_bias,
     const float* __restrict__ d_skip, float* __restrict__ state, const int* __restrict__ rec_slots,
@@ -159,13 +159,13 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(
   __syncthreads();
   float y[4] = {0.f, 0.f, 0.f, 0.f};
   if (on) {
-    constexpr int ROWS = 8;
+    constexpr int ROWS = 4;
     for (int n0 = r0; n0 < N; n0 += rg * ROWS) {
       float4 S[ROWS];
 #pragma unroll
       for (int k = 0; k < ROWS; ++k) {
         const int n = n0 + k * rg;
-        S[k] = (carried && n < N) ? *reinterpret_cast<const float4*>(st + (size_t)n * V + col)
+        S[k] = (carried && n < N) ? __ldcs(reinterpret_cast<const float4*>(st + (size_t)n * V + col))
                                   : make_float4(0.f, 0.f, 0.f, 0.f);
       }
 #pragma unroll
@@ -181,7 +181,7 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(
           y[1] = fmaf(S[k].y, cn, y[1]);
           y[2] = fmaf(S[k].z, cn, y[2]);
           y[3] = fmaf(S[k].w, cn, y[3]);
-          if (st != nullptr) *reinterpret_cast<float4*>(st + (size_t)n * V + col) = S[k];
+          if (st != nullptr) __stcs(reinterpret_cast<float4*>(st + (size_t)n * V + col), S[k]);
         }
       }
     }

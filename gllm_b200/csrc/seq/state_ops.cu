@@ -360,13 +360,15 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ o, int n, cons
   }
 }
 
+// `block` > 0: gate and up columns alternate in blocks of that many (the layout of the tcgen05 GEMM's gated epilogue)
 template <typename T>
 __global__ void silu_mul_kernel(const T* __restrict__ gu, long ld, int F, T* __restrict__ out, long ldo,
-                                size_t total) {
+                                size_t total, int block) {
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= total) return;
   const size_t t = i / F, f = i - t * F;
-  out[t * ldo + f] = from_f<T>(silu_f(to_f(gu[t * ld + f])) * to_f(gu[t * ld + F + f]));
+  const size_t g = block > 0 ? f / block * (2 * block) + f % block : f, u = block > 0 ? g + block : F + f;
+  out[t * ldo + f] = from_f<T>(silu_f(to_f(gu[t * ld + g])) * to_f(gu[t * ld + u]));
 }
 
 // Router logits for small batches: one warp per (token, expert), lanes over the width in a fixed order, fp32 result.
@@ -783,14 +785,15 @@ GLLM_EXPORT int gllm_seq_gated_group_norm(const void* o, int n, const void* gate
 }
 
 GLLM_EXPORT int gllm_seq_silu_mul(const void* gu, long ld, int ntok, int F, void* out, long ldo, int is_f32,
-                                  void* stream) {
+                                  int block, void* stream) {
   if (ntok <= 0 || F <= 0) return 0;
+  if (block > 0 && F % block != 0) return 2;
   cudaStream_t st = (cudaStream_t)stream;
   const size_t total = (size_t)ntok * F;
   const unsigned blocks = (unsigned)((total + 255) / 256);
   GLLM_BY_DTYPE(is_f32,
-                (silu_mul_kernel<bf16_t><<<blocks, 256, 0, st>>>((const bf16_t*)gu, ld, F, (bf16_t*)out, ldo, total)),
-                (silu_mul_kernel<float><<<blocks, 256, 0, st>>>((const float*)gu, ld, F, (float*)out, ldo, total)));
+                (silu_mul_kernel<bf16_t><<<blocks, 256, 0, st>>>((const bf16_t*)gu, ld, F, (bf16_t*)out, ldo, total, block)),
+                (silu_mul_kernel<float><<<blocks, 256, 0, st>>>((const float*)gu, ld, F, (float*)out, ldo, total, block)));
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
 }

@@ -228,12 +228,13 @@ def gated_group_norm(o, gate, w, group, eps, act, out_scale=1.0, out=None, out_d
     return fn(o, gate, w, group, eps, act, out_scale, out, out_dtype)
 
 
-def silu_mul(gu, out=None):
+def silu_mul(gu, out=None, block=0):
+    """silu(gate) * up of [gate | up] rows; `block` > 0: blocks of that many gate and up columns alternate."""
     if gu.is_cuda:
-        if gu.dtype == torch.bfloat16 and gu.is_contiguous() and out is None:
+        if gu.dtype == torch.bfloat16 and gu.is_contiguous() and out is None and not block:
             return _sm().silu_and_mul(gu)
-        return _seq().silu_mul(gu, out)
-    return ref.silu_mul(gu) if out is None else out.copy_(ref.silu_mul(gu))
+        return _seq().silu_mul(gu, out, block)
+    return ref.silu_mul(gu, block) if out is None else out.copy_(ref.silu_mul(gu, block))
 
 
 def router_topk(h, w, top_k):

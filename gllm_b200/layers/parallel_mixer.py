@@ -7,10 +7,12 @@ projections' biases in its epilogue, for cores that have them), each core
 writes scale_i * result_i into its column slice of one buffer, ONE output GEMM over the concatenated output
 projections — sum_i scale_i * o_i(core_i(h)). With a single core it is the plain mixer.
 
-`GatedBranch` is a gated feed-forward as one more branch of the same sum: it reads the same input through its own
-gate / up product (whose epilogue forms silu(gate) * up) and writes its columns of the joint buffer, so a block whose
-mixer and feed-forward run side by side has one output GEMM, mixer(h) + ff(h) = [core(h) | act(h)] [W_o | W_down]^T,
-summed in the accumulator.
+A gated feed-forward can be one more branch of the same sum (`ff`): silu(gate h) * (up h) fills its own columns of the
+joint buffer, so a block whose mixer and feed-forward run side by side has one output GEMM,
+mixer(h) + ff(h) = [core(h) | act(h)] [W_o | W_down]^T, summed in the accumulator. Its gate and up rows follow the cores'
+rows in the input weight. Small batches (decode) run ONE input GEMM over all rows and a small activation kernel; larger
+ones run the cores' rows and the gate / up rows apart, the latter with the tcgen05 GEMM's SiLU-gate epilogue (rows
+interleaved per 128; bf16 on CUDA with ff % 128 == 0).
 """
 from __future__ import annotations
 
@@ -22,29 +24,7 @@ from torch import nn
 from gllm_b200.layers import functional as Fn
 
 
-class GatedBranch(nn.Module):
-    """silu(gate h) * (up h) into a column slice; the down projection is part of the mixer's joint output weight. On
-    CUDA in bf16 with ff % 128 == 0 gate and up rows are interleaved per 128 and the product is the tcgen05 GEMM's
-    SiLU-gate epilogue."""
-
-    def __init__(self, hidden: int, ff: int, dtype, device, align: int = 8):
-        super().__init__()
-        self.ff = ff
-        self.fused = torch.device(device).type == "cuda" and dtype == torch.bfloat16 and ff % 128 == 0 and \
-            hidden % 8 == 0 and align % 8 == 0
-        self.gate_up_w = nn.Parameter(torch.zeros(2 * ff, hidden, dtype=dtype, device=device), requires_grad=False)
-
-    def load(self, gate, up):
-        from gllm_b200.ops import ref
-        gu = torch.cat([gate, up], 0)
-        assert tuple(gu.shape) == tuple(self.gate_up_w.shape), (tuple(gu.shape), tuple(self.gate_up_w.shape))
-        self.gate_up_w.data.copy_(ref.interleave_gate_up(gu, 128) if self.fused else gu)
-
-    def act(self, h, out):
-        if self.fused:
-            Fn.linear_silu_mul(h, self.gate_up_w, out)
-        else:
-            Fn.silu_mul(Fn.linear_any(h, self.gate_up_w), out)
+_JOINT_INPUT_MAX_TOKENS = 128      # up to here one launch less is worth more than the fused activation
 
 
 class CoreMixer(nn.Module):
@@ -56,10 +36,13 @@ class CoreMixer(nn.Module):
         self.n_in = sum(c.n_in for c in cores)
         self.n_out = sum(c.n_out for c in cores)
         # a parallel feed-forward: `ff` more columns of the joint buffer (its slice starts at a multiple of 8)
-        self.ff_at = (self.n_out + 7) // 8 * 8
-        self.ff = GatedBranch(hidden, ff, dtype, device, (self.ff_at + ff) % 8 or 8) if ff else None
-        self.n_joint = self.ff_at + ff if ff else self.n_out
-        n_in_pad = (self.n_in + 7) // 8 * 8            # the tensor-core GEMM wants N % 8 == 0; pad rows stay zero
+        self.ff, self.ff_at = int(ff), (self.n_out + 7) // 8 * 8
+        self.n_joint = self.ff_at + self.ff if ff else self.n_out
+        self.ff_block = 128 if torch.device(device).type == "cuda" and dtype == torch.bfloat16 and ff and \
+            ff % 128 == 0 and hidden % 8 == 0 else 0
+        # the tensor-core GEMM wants N % 8 == 0; pad rows stay zero
+        self.n_in_pad = (self.n_in + 7) // 8 * 8
+        n_in_pad = self.n_in_pad + 2 * self.ff
         self.in_w = nn.Parameter(torch.zeros(n_in_pad, hidden, dtype=dtype, device=device), requires_grad=False)
         self.o_w = nn.Parameter(torch.zeros(hidden, self.n_joint, dtype=dtype, device=device), requires_grad=False)
         # biases of the input projection ('<projection>.b'), for cores that declare `has_bias`; rows of others stay 0
@@ -77,12 +60,16 @@ class CoreMixer(nn.Module):
         return {"kind": "multi", "kv": kv[0] if kv else None, "rec": rec[0] if rec else None}
 
     def forward(self, inp, h: torch.Tensor, cache, run_id: int) -> torch.Tensor:
-        proj = Fn.linear_any(h, self.in_w, self.in_b)
         joint = torch.empty(h.shape[0], self.n_joint, dtype=h.dtype, device=h.device)
-        if self.ff is not None:
-            if self.ff_at > self.n_out:
-                joint[:, self.n_out:self.ff_at].zero_()        # meets zero weight columns, must be finite
-            self.ff.act(h, joint[:, self.ff_at:])
+        if self.ff and self.ff_at > self.n_out:
+            joint[:, self.n_out:self.ff_at].zero_()            # meets zero weight columns, must be finite
+        if self.ff_block and h.shape[0] > _JOINT_INPUT_MAX_TOKENS and self.in_b is None:
+            proj = Fn.linear_any(h, self.in_w[:self.n_in_pad])
+            Fn.linear_silu_mul(h, self.in_w[self.n_in_pad:], joint[:, self.ff_at:])
+        else:
+            proj = Fn.linear_any(h, self.in_w, self.in_b)
+            if self.ff:
+                Fn.silu_mul(proj[:, self.n_in_pad:], joint[:, self.ff_at:], self.ff_block)
         ci = co = 0
         for c, s in zip(self.cores, self.scales):
             c.core(inp, proj[:, ci:ci + c.n_in], cache, run_id, joint[:, co:co + c.n_out], s)
@@ -108,9 +95,11 @@ class CoreMixer(nn.Module):
             c.load_extra(reader, p, put)
         w = torch.cat(rows, 0)
         self.in_w.data[: w.shape[0]].copy_(w)
-        if self.ff is None:
+        if not self.ff:
             put(self.o_w, torch.cat(cols, 1))
             return
-        self.ff.load(reader.get(ff_pre + "gate"), reader.get(ff_pre + "up"))
+        from gllm_b200.ops import ref
+        gu = torch.cat([reader.get(ff_pre + "gate"), reader.get(ff_pre + "up")], 0)
+        put(self.in_w.data[self.n_in_pad:], ref.interleave_gate_up(gu, self.ff_block) if self.ff_block else gu)
         put(self.o_w.data[:, :self.n_out], torch.cat(cols, 1))
         put(self.o_w.data[:, self.ff_at:], reader.get(ff_pre + "down"))

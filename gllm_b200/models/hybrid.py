@@ -58,7 +58,7 @@ The parallel form (mult: the residual multiplier; one norm feeds both sublayers;
     loop: the span's passes follow each other, each with its own cache entries; nothing happens in between
     logits = head @ (rms(x) * final_norm)
 
-Here mixer and feed-forward share one output GEMM (`CoreMixer` with a `GatedBranch`), so the stream update is
+Here mixer and feed-forward share one output GEMM (`CoreMixer` with `ff`), so the stream update is
 x += mult * y in one kernel that also emits x in the compute dtype for G; the second update (norm of the side branch,
 multiplier, next layer's norm1) is one kernel as in the sandwich form.
 

@@ -871,9 +871,11 @@ def gelu_gate_embed(g: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, col
     return (F.gelu(g.float(), approximate="tanh") * e.float()).to(g.dtype)
 
 
-def silu_mul(gu: torch.Tensor) -> torch.Tensor:
-    """gu [T, 2F] = [gate | up] -> silu(gate) * up."""
+def silu_mul(gu: torch.Tensor, block: int = 0) -> torch.Tensor:
+    """gu [T, 2F] = [gate | up] -> silu(gate) * up. `block` > 0: blocks of gate and up columns alternate."""
     f = gu.shape[1] // 2
+    if block:
+        gu = gu.reshape(gu.shape[0], f // block, 2, block).transpose(1, 2).reshape(gu.shape[0], 2 * f)
     return (F.silu(gu[:, :f].float()) * gu[:, f:].float()).to(gu.dtype)
 
 

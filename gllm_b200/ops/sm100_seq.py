@@ -38,7 +38,7 @@ def _L():
             "gllm_seq_key_decay": [P, G, P, F, P, I, I, I, P],
             "gllm_seq_gemm_mma_f32out": [P, G, G, P, G, G, P, G, G, I, I, I, I, P],
             "gllm_seq_gated_group_norm": [P, I, P, G, P, I, I, F, I, F, P, G, I, I, P],
-            "gllm_seq_silu_mul": [P, G, I, I, P, G, I, P],
+            "gllm_seq_silu_mul": [P, G, I, I, P, G, I, I, P],
             "gllm_seq_router_select": [P, I, I, I, P, P, P],
             "gllm_seq_router_logits": [P, G, P, I, I, I, P, I, P],
             "gllm_seq_router_logits_mma": [P, G, P, I, I, I, P, P],
@@ -341,11 +341,12 @@ def gated_group_norm(o, gate, w, group, eps, act, out_scale=1.0, out=None, out_d
     return out
 
 
-def silu_mul(gu, out=None):
+def silu_mul(gu, out=None, block: int = 0):
+    """gu [T, 2F] = [gate | up], or with `block` alternating blocks of gate and up columns."""
     t, f = gu.shape[0], gu.shape[1] // 2
     out = torch.empty(t, f, dtype=gu.dtype, device=gu.device) if out is None else out
     assert gu.stride(1) == 1 and out.stride(1) == 1 and out.shape == (t, f) and out.dtype == gu.dtype
-    check(_L().gllm_seq_silu_mul(_p(gu), gu.stride(0), t, f, _p(out), out.stride(0), _f32(gu), stream_ptr()),
+    check(_L().gllm_seq_silu_mul(_p(gu), gu.stride(0), t, f, _p(out), out.stride(0), _f32(gu), int(block), stream_ptr()),
           "seq_silu_mul")
     sm100._count()
     return out
