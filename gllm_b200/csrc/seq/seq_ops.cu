@@ -338,10 +338,10 @@ __global__ void conv_silu_kernel(const T* __restrict__ xz, long ldxz, int C, con
   out[(size_t)t * C + c] = from_f<T>(act == 0 ? acc / (1.0f + expf(-acc)) : acc);
 }
 
-// The same convolution for bf16 rows whose channels come in aligned groups of 8: a thread owns 8 channels (16-byte loads
-// and stores, weights in registers) and walks `rows` consecutive batch rows with the last TAPS - 1 inputs in
-// registers, so every input row is read once per block instead of TAPS times. The next row's load is in flight while
-// the current one is computed. Sequences of one token also update their carried inputs here (longer ones: the kernel
+// The same convolution for bf16 rows whose channels come in aligned groups of 4: a thread owns 4 channels (8-byte loads
+// and stores, weights in registers: 8 channels would halve the occupancy) and walks `rows` consecutive batch rows with
+// the last TAPS - 1 inputs in registers, so every input row is read once per block instead of TAPS times. The next
+// row's load is in flight while the current one is computed. Sequences of one token also update their carried inputs here (longer ones: the kernel
 // below, after every block has read them).
 template <int TAPS>
 __global__ void __launch_bounds__(128) conv_silu_vec_kernel(
@@ -349,31 +349,30 @@ __global__ void __launch_bounds__(128) conv_silu_vec_kernel(
     __nv_bfloat16* __restrict__ state, const int* __restrict__ rec_slots, const int* __restrict__ seq_lens,
     const int* __restrict__ qsl, int nseq, int ntok, int rows, __nv_bfloat16* __restrict__ out, int act,
     const float* __restrict__ in_bias) {
-  const int c = (blockIdx.y * 128 + threadIdx.x) * 8;
+  const int c = (blockIdx.y * 128 + threadIdx.x) * 4;
   if (c >= C) return;
   const int t0 = blockIdx.x * rows, t1 = min(t0 + rows, ntok);
-  __align__(16) float wr[8 * TAPS], br[8], ib[8];              // weight of channel e, tap j: wr[e * TAPS + j]
+  __align__(16) float wr[4 * TAPS], br[4], ib[4];              // weight of channel e, tap j: wr[e * TAPS + j]
 #pragma unroll
-  for (int e = 0; e < 8 * TAPS; e += 4)
+  for (int e = 0; e < 4 * TAPS; e += 4)
     *reinterpret_cast<float4*>(wr + e) = *reinterpret_cast<const float4*>(w + (size_t)c * TAPS + e);
+  *reinterpret_cast<float4*>(br) = *reinterpret_cast<const float4*>(b + c);
 #pragma unroll
-  for (int e = 0; e < 8; e += 4) *reinterpret_cast<float4*>(br + e) = *reinterpret_cast<const float4*>(b + c + e);
-#pragma unroll
-  for (int e = 0; e < 8; ++e) ib[e] = in_bias != nullptr ? in_bias[c + e] : 0.f;
-  auto unpack = [](const uint4 v, float (&f)[8]) {
+  for (int e = 0; e < 4; ++e) ib[e] = in_bias != nullptr ? in_bias[c + e] : 0.f;
+  auto unpack = [](const uint2 v, float (&f)[4]) {
     const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&v);
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
+    for (int e = 0; e < 2; ++e) {
       const float2 p = __bfloat1622float2(h[e]);
       f[2 * e] = p.x;
       f[2 * e + 1] = p.y;
     }
   };
-  float win[TAPS][8];                            // win[0 .. TAPS-2]: inputs before the row; win[TAPS-1]: the row's own
+  float win[TAPS][4];                            // win[0 .. TAPS-2]: inputs before the row; win[TAPS-1]: the row's own
   int s = find_seq(qsl, nseq, t0), q0 = 0, q1 = -1;
-  uint4 cur = *reinterpret_cast<const uint4*>(xz + (size_t)t0 * ldxz + c);
+  uint2 cur = *reinterpret_cast<const uint2*>(xz + (size_t)t0 * ldxz + c);
   for (int t = t0; t < t1; ++t) {
-    const uint4 nxt = t + 1 < t1 ? *reinterpret_cast<const uint4*>(xz + (size_t)(t + 1) * ldxz + c) : cur;
+    const uint2 nxt = t + 1 < t1 ? *reinterpret_cast<const uint2*>(xz + (size_t)(t + 1) * ldxz + c) : cur;
     if (t >= q1) {                               // first row of the block or of a sequence: gather its past
       while (s + 1 < nseq && qsl[s + 1] <= t) ++s;
       q0 = qsl[s];
@@ -384,18 +383,18 @@ __global__ void __launch_bounds__(128) conv_silu_vec_kernel(
       for (int j = 0; j < TAPS - 1; ++j) {
         const int src = li - (TAPS - 1) + j;
         const bool own = src >= 0, have = own || (carried && pos0 + src >= 0);
-        float f[8];
-        if (own) unpack(*reinterpret_cast<const uint4*>(xz + (size_t)(q0 + src) * ldxz + c), f);
+        float f[4];
+        if (own) unpack(*reinterpret_cast<const uint2*>(xz + (size_t)(q0 + src) * ldxz + c), f);
         else if (have)
-          unpack(*reinterpret_cast<const uint4*>(state + ((size_t)rec_slots[s] * (TAPS - 1) + TAPS - 1 + src) * C + c), f);
+          unpack(*reinterpret_cast<const uint2*>(state + ((size_t)rec_slots[s] * (TAPS - 1) + TAPS - 1 + src) * C + c), f);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) win[j][e] = have ? f[e] + ib[e] : 0.f;
+        for (int e = 0; e < 4; ++e) win[j][e] = have ? f[e] + ib[e] : 0.f;
       }
     }
     unpack(cur, win[TAPS - 1]);
-    __align__(16) __nv_bfloat16 o[8];
+    __align__(16) __nv_bfloat16 o[4];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) {
+    for (int e = 0; e < 4; ++e) {
       win[TAPS - 1][e] += ib[e];
       float acc = br[e];
 #pragma unroll
@@ -404,16 +403,16 @@ __global__ void __launch_bounds__(128) conv_silu_vec_kernel(
 #pragma unroll
       for (int j = 0; j + 1 < TAPS; ++j) win[j][e] = win[j + 1][e];
     }
-    *reinterpret_cast<uint4*>(out + (size_t)t * C + c) = *reinterpret_cast<const uint4*>(o);
+    *reinterpret_cast<uint2*>(out + (size_t)t * C + c) = *reinterpret_cast<const uint2*>(o);
     if (TAPS > 1 && state != nullptr && q1 - q0 == 1) {
       // a single token's sequence: nobody else reads its slot, so the carried inputs move up here
       __nv_bfloat16* st = state + (size_t)rec_slots[s] * (TAPS - 1) * C + c;
       const bool carried = seq_lens[s] > 1;
 #pragma unroll
       for (int j = 0; j + 1 < TAPS - 1; ++j)
-        *reinterpret_cast<uint4*>(st + (size_t)j * C) =
-            carried ? *reinterpret_cast<const uint4*>(st + (size_t)(j + 1) * C) : make_uint4(0u, 0u, 0u, 0u);
-      *reinterpret_cast<uint4*>(st + (size_t)(TAPS - 2) * C) = cur;
+        *reinterpret_cast<uint2*>(st + (size_t)j * C) =
+            carried ? *reinterpret_cast<const uint2*>(st + (size_t)(j + 1) * C) : make_uint2(0u, 0u);
+      *reinterpret_cast<uint2*>(st + (size_t)(TAPS - 2) * C) = cur;
     }
     cur = nxt;
   }
@@ -716,11 +715,11 @@ GLLM_EXPORT int gllm_seq_conv_silu(const void* xz, long ldxz, int ntok, int nseq
                                                              (const int*)rec_slots, (const int*)seq_lens,
                                                              (const int*)qsl, 1);
   } else {
-    const bool vec = C % 8 == 0 && ldxz % 8 == 0 && ((uintptr_t)xz & 15) == 0 && taps >= 1 && taps <= 4 &&
-                     ((uintptr_t)state & 15) == 0 && ((uintptr_t)out & 15) == 0 && ((uintptr_t)w & 15) == 0 &&
+    const bool vec = C % 4 == 0 && ldxz % 4 == 0 && ((uintptr_t)xz & 7) == 0 && taps >= 1 && taps <= 4 &&
+                     ((uintptr_t)state & 7) == 0 && ((uintptr_t)out & 7) == 0 && ((uintptr_t)w & 15) == 0 &&
                      ((uintptr_t)b & 15) == 0;
     const int rows = ntok >= 2048 ? 16 : (ntok >= 512 ? 4 : 1);
-    dim3 vgrid((ntok + rows - 1) / rows, (C / 8 + 127) / 128);
+    dim3 vgrid((ntok + rows - 1) / rows, (C / 4 + 127) / 128);
 #define GLLM_CONV_VEC(TAPS)                                                                                        \
   conv_silu_vec_kernel<TAPS><<<vgrid, 128, 0, st>>>(                                                               \
       (const __nv_bfloat16*)xz, ldxz, C, (const float*)w, (const float*)b, (__nv_bfloat16*)state,                  \

@@ -99,9 +99,10 @@ def _require_kernels(model_dir: str):
             cfg = json.load(f)
     except OSError:
         return
-    if cfg.get("architecture") in ("Saritar", "Femolix", "Bevovik", "Notadra", "Vikupel"):
+    arch = cfg.get("architecture")
+    if arch in ("Saritar", "Femolix", "Bevovik", "Notadra", "Vikupel"):
         from gllm_b200.ops import lib
-        lib.require({"seq", "gemm", "attn", "moe"})
+        lib.require({"seq", "gemm", "attn"} | (set() if arch == "Vikupel" else {"moe"}))
 
 
 def main(argv=None) -> int:
