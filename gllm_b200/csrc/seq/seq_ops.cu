@@ -718,7 +718,7 @@ GLLM_EXPORT int gllm_seq_conv_silu(const void* xz, long ldxz, int ntok, int nseq
     const bool vec = C % 4 == 0 && ldxz % 4 == 0 && ((uintptr_t)xz & 7) == 0 && taps >= 1 && taps <= 4 &&
                      ((uintptr_t)state & 7) == 0 && ((uintptr_t)out & 7) == 0 && ((uintptr_t)w & 15) == 0 &&
                      ((uintptr_t)b & 15) == 0;
-    const int rows = ntok >= 2048 ? 16 : (ntok >= 512 ? 4 : 1);
+    const int rows = ntok >= 2048 ? 16 : (ntok >= 512 ? 8 : 1);
     dim3 vgrid((ntok + rows - 1) / rows, (C / 4 + 127) / 128);
 #define GLLM_CONV_VEC(TAPS)                                                                                        \
   conv_silu_vec_kernel<TAPS><<<vgrid, 128, 0, st>>>(                                                               \
