@@ -140,7 +140,7 @@ def test_gate_norm_token_side_stream_update(dt, tol):
 
 
 ATT = [  # heads, kv heads, dim, vdim, window, page size
-    (4, 2, 64, 64, 20, 16), (8, 2, 128, 128, 100, 16), (6, 2, 64, 64, None, 8), (8, 8, 128, 128, None, 16),
+    (4, 2, 64, 64, 20, 16), (8, 2, 128, 128, 100, 16), (6, 1, 64, 64, None, 8), (8, 8, 128, 128, None, 16),
     (4, 1, 256, 256, 33, 16), (6, 3, 48, 40, 17, 16), (5, 1, 64, 32, None, 16), (16, 1, 64, 64, 130, 64),
     (4, 4, 128, 128, 1, 16)]
 
