@@ -91,6 +91,7 @@ __device__ __forceinline__ float tanh_exp(float x) { return 1.0f - __fdividef(2.
 
 // Options that some designs add to the masked attention (all of them optional):
 //   r1, r2 [Hq]     distance bias: r1 ln(1 + r2 (i - j)) is taken off the scaled score of key j for the query at i
+//   dtab [n, Hq]    distance table (fp32): row min(i - j, n - 1) is added to the scaled score
 //   v_turn [tok, D] cos | sin (fp32) of the query's position: the values were rotated by their own positions, every
 //                   head's result is turned back by the query's (entry m with m + D / 2)
 //   gate            [tok, Hq * D] rows of stride ldg: the result is multiplied by sigmoid(gate), last
@@ -100,21 +101,30 @@ struct AttnExtras {
   const __nv_bfloat16* gate = nullptr;
   int64_t ldg = 0;
   const float* v_turn = nullptr;
-  bool any() const { return r1 != nullptr || gate != nullptr || v_turn != nullptr; }
+  const float* dtab = nullptr;
+  int dtab_n = 0;
+  bool any() const { return r1 != nullptr || gate != nullptr || v_turn != nullptr || dtab != nullptr; }
 };
-inline AttnExtras make_extras(const void* r1, const void* r2, const void* gate, int64_t ldg, const void* v_turn) {
+inline AttnExtras make_extras(const void* r1, const void* r2, const void* gate, int64_t ldg, const void* v_turn,
+                              const void* dtab, int dtab_n) {
   AttnExtras e;
   e.r1 = reinterpret_cast<const float*>(r1);
   e.r2 = reinterpret_cast<const float*>(r2);
   e.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
   e.ldg = ldg;
   e.v_turn = reinterpret_cast<const float*>(v_turn);
+  e.dtab = reinterpret_cast<const float*>(dtab);
+  e.dtab_n = dtab_n;
   return e;
 }
 
 // the distance bias in the base-2 domain of the softmax: r1 ln(.) log2(e) = r1 log2(.)
 __device__ __forceinline__ float dist_bias_log2(float r1, float r2, int dist) {
   return r1 * __log2f(fmaf(r2, (float)max(dist, 0), 1.0f));
+}
+// the distance table in the base-2 domain: the entry of distance `dist` for one head (tab points at its column)
+__device__ __forceinline__ float dist_table_log2(const float* tab, int n, int Hq, int dist) {
+  return __ldg(tab + static_cast<size_t>(min(max(dist, 0), n - 1)) * Hq) * 1.4426950408889634f;
 }
 __device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
 

@@ -38,6 +38,8 @@ struct MlaParams {
   const int32_t* positions;   // [tokens] absolute position of the token (kv_len = position + 1)
   int max_blocks, H, page_size, num_splits;
   float scale_log2;
+  int window;                 // a token at position i sees keys j with i - j < window (0: the whole past)
+  const float* sink;          // [H] one more logit per head in the denominator, without a value (null: none)
 };
 
 __global__ void __launch_bounds__(kAttnThreads)
@@ -60,8 +62,10 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmap, const MlaParams p) {
   const int seq = p.tok_seq != nullptr ? p.tok_seq[tok] : tok;
   const int kv_len = p.positions[tok] + 1;
   const int n_tiles = (kv_len + kTileN - 1) / kTileN;
-  const int tps = (n_tiles + p.num_splits - 1) / p.num_splits;
-  const int tile_begin = min(split * tps, n_tiles);
+  const int win_lo = p.window > 0 ? max(0, kv_len - p.window) : 0;          // first visible key
+  const int tile_lo = win_lo / kTileN;
+  const int tps = (n_tiles - tile_lo + p.num_splits - 1) / p.num_splits;
+  const int tile_begin = min(tile_lo + split * tps, n_tiles);
   const int tile_end = min(tile_begin + tps, n_tiles);
   const int page_bytes = p.page_size * kLat * 2;
   const int n_rows = min(16, p.H - hbase);
@@ -156,7 +160,7 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmap, const MlaParams p) {
       for (int e = 0; e < 4; ++e) {
         const int col = abs0 + nt * 8 + (e & 1);
         float v = sc[nt][e] * p.scale_log2;
-        if (col >= kv_len) v = -INFINITY;
+        if (col >= kv_len || col < win_lo) v = -INFINITY;
         sc[nt][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
       }
@@ -240,7 +244,10 @@ mla_attn_kernel(const __grid_constant__ CUtensorMap tmap, const MlaParams p) {
   for (int r = 0; r < 2; ++r) {
     const int row = g + r * 8;
     if (row >= n_rows) continue;
-    const float l_all = red_sum[row] + red_sum[16 + row] + red_sum[32 + row] + red_sum[48 + row];
+    float l_all = red_sum[row] + red_sum[16 + row] + red_sum[32 + row] + red_sum[48 + row];
+    // the sink joins the first split (which always has a key): its weight then carries it through the merge
+    if (p.sink != nullptr && split == 0 && m_run[r] > -INFINITY)
+      l_all += exp2f(p.sink[hbase + row] * 1.4426950408889634f - m_run[r]);
     const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
     const size_t th = static_cast<size_t>(tok) * p.H + hbase + row;
 #pragma unroll
@@ -308,10 +315,11 @@ using namespace b200;
 
 // q [tokens, H, 576] bf16 contiguous -> out [tokens, H, 512]; cache = latent pages [num_pages, 1, 9, page, 64].
 // part_o / part_lse are only touched when num_splits > 1.
+// window (0: none) and sink (null: none): see MlaParams.
 GLLM_EXPORT int gllm_mla_attention(const void* q, void* out, const void* cache, int64_t num_pages,
                                    const void* block_table, const void* tok_seq, const void* positions, void* part_o,
                                    void* part_lse, int tokens, int max_blocks, int H, int page_size, int num_splits,
-                                   float scale, void* stream) {
+                                   float scale, int window, const void* sink, void* stream) {
   if (tokens <= 0) return 0;
   if (page_size < 8 || kTileN % page_size != 0) {
     fprintf(stderr, "[gllm_b200] mla_attention: unsupported page_size=%d\n", page_size);
@@ -330,6 +338,8 @@ GLLM_EXPORT int gllm_mla_attention(const void* q, void* out, const void* cache, 
   p.max_blocks = max_blocks; p.H = H; p.page_size = page_size;
   p.num_splits = num_splits < 1 ? 1 : num_splits;
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.window = window;
+  p.sink = reinterpret_cast<const float*>(sink);
   static PerDeviceOnce configured;
   if (configured.need()) {
     CUDA_CHECK_RET(cudaFuncSetAttribute(mla_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kMlaSmem));

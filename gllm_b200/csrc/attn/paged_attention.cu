@@ -163,6 +163,15 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_cons
     for (int r = 0; r < 2; ++r)
       if (g + 8 * r < p.GP) { b1[r] = p.ex.r1[hbase + g + 8 * r]; b2[r] = p.ex.r2[hbase + g + 8 * r]; }
   }
+  const float* tab[2] = {nullptr, nullptr};          // distance table columns of the two heads, and their far entries
+  float far[2] = {0.f, 0.f};
+  if (EX && p.ex.dtab != nullptr) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      tab[r] = p.ex.dtab + hbase + (g + 8 * r < p.GP ? g + 8 * r : 0);
+      far[r] = dist_table_log2(tab[r], p.ex.dtab_n, p.Hq, p.ex.dtab_n - 1);
+    }
+  }
 
   uint32_t it = 0;
   for (int tile = tile_begin; tile < tile_end; ++tile, ++it) {
@@ -191,6 +200,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_cons
     }
     // mask + online softmax (rows g and g+8)
     const int abs0 = tile * kTileN + tok0 + 2 * t;
+    const bool far_tile = EX && seq_len - (tile + 1) * kTileN >= p.ex.dtab_n - 1;    // every key at the table's end
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt) {
@@ -198,7 +208,9 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_cons
       for (int e = 0; e < 4; ++e) {
         const int col = abs0 + nt * 8 + (e & 1);
         float v = p.cap_log2 > 0.f ? p.cap_log2 * tanh_exp(sc[nt][e] * p.scale_over_cap) : sc[nt][e] * p.scale_log2;
-        if (EX) v -= dist_bias_log2(b1[e >> 1], b2[e >> 1], seq_len - 1 - col);
+        if (EX && p.ex.r1 != nullptr) v -= dist_bias_log2(b1[e >> 1], b2[e >> 1], seq_len - 1 - col);
+        if (EX && p.ex.dtab != nullptr)
+          v += far_tile ? far[e >> 1] : dist_table_log2(tab[e >> 1], p.ex.dtab_n, p.Hq, seq_len - 1 - col);
         if (col >= seq_len || col < win_lo) v = -INFINITY;
         sc[nt][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -480,6 +492,15 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
 #pragma unroll
     for (int r = 0; r < 2; ++r) { b1[r] = p.ex.r1[r_head[r]]; b2[r] = p.ex.r2[r_head[r]]; }
   }
+  const float* tab[2] = {nullptr, nullptr};          // distance table columns of the two rows' heads, and their far entries
+  float far[2] = {0.f, 0.f};
+  if (EX && p.ex.dtab != nullptr) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      tab[r] = p.ex.dtab + r_head[r];
+      far[r] = dist_table_log2(tab[r], p.ex.dtab_n, p.Hq, p.ex.dtab_n - 1);
+    }
+  }
 
   uint32_t it = 0;
   for (int tile = tile_lo; tile < n_tiles; ++tile, ++it) {
@@ -505,6 +526,8 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
       }
     }
     const int abs0 = tile * kTileN + 2 * t;
+    // every key of the tile at the table's end, for every row of the block
+    const bool far_tile = EX && ctx_len + tok_base - ((tile + 1) * kTileN - 1) >= p.ex.dtab_n - 1;
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int nt = 0; nt < 8; ++nt) {
@@ -512,7 +535,9 @@ attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_con
       for (int e = 0; e < 4; ++e) {
         const int col = abs0 + nt * 8 + (e & 1);
         float v = p.cap_log2 > 0.f ? p.cap_log2 * tanh_exp(sc[nt][e] * p.scale_over_cap) : sc[nt][e] * p.scale_log2;
-        if (EX) v -= dist_bias_log2(b1[e >> 1], b2[e >> 1], lim[e >> 1] - col);
+        if (EX && p.ex.r1 != nullptr) v -= dist_bias_log2(b1[e >> 1], b2[e >> 1], lim[e >> 1] - col);
+        if (EX && p.ex.dtab != nullptr)
+          v += far_tile ? far[e >> 1] : dist_table_log2(tab[e >> 1], p.ex.dtab_n, p.Hq, lim[e >> 1] - col);
         if (col > lim[e >> 1] || col < clo[e >> 1] || (p.window > 0 && col <= lim[e >> 1] - p.window)) v = -INFINITY;
         sc[nt][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -826,10 +851,10 @@ GLLM_EXPORT int gllm_attn_decode_mask(const void* q, int64_t q_ts, void* out, in
                                       int Hkv, int D, int page_size, float scale, int window, int chunk,
                                       const void* sink, float out_scale, float softcap, const void* r1,
                                       const void* r2, const void* gate, int64_t ldg, const void* v_turn,
-                                      void* stream) {
+                                      const void* dtab, int dtab_n, void* stream) {
   return attn_decode_impl(q, q_ts, out, k_cache, v_cache, num_pages, block_table, seq_lens, nullptr, nullptr,
                           num_seqs, seq_offset, max_blocks, Hq, Hkv, D, page_size, 1, scale, nullptr, stream, window,
-                          sink, chunk, out_ts, out_scale, softcap, make_extras(r1, r2, gate, ldg, v_turn));
+                          sink, chunk, out_ts, out_scale, softcap, make_extras(r1, r2, gate, ldg, v_turn, dtab, dtab_n));
 }
 
 GLLM_EXPORT int gllm_attn_prefill_mask(const void* q, int64_t q_ts, void* out, int64_t out_ts, const void* k_cache,
@@ -838,8 +863,8 @@ GLLM_EXPORT int gllm_attn_prefill_mask(const void* q, int64_t q_ts, void* out, i
                                        int max_q_len, int max_blocks, int Hq, int Hkv, int D, int page_size,
                                        float scale, int window, int chunk, const void* sink, float out_scale,
                                        float softcap, const void* r1, const void* r2, const void* gate, int64_t ldg,
-                                       const void* v_turn, void* stream) {
+                                       const void* v_turn, const void* dtab, int dtab_n, void* stream) {
   return attn_prefill_impl(q, q_ts, out, k_cache, v_cache, num_pages, block_table, seq_lens, q_start, num_seqs,
                            seq_offset, max_q_len, max_blocks, Hq, Hkv, D, page_size, scale, stream, window, sink,
-                           chunk, out_ts, out_scale, softcap, make_extras(r1, r2, gate, ldg, v_turn));
+                           chunk, out_ts, out_scale, softcap, make_extras(r1, r2, gate, ldg, v_turn, dtab, dtab_n));
 }

@@ -50,20 +50,28 @@ struct TcAttnParams {
   const float* sink;
   int64_t out_ts;     // output row stride (elements)
   int window;         // sliding window: a query at i sees keys j with i - j < window (0 = the whole past)
-  AttnExtras ex;      // distance bias (kernel template BIAS), turned values, output gate
+  AttnExtras ex;      // distance bias or table (kernel template BIAS), turned values, output gate
   uint32_t v_lbo16, v_sbo16, v_kadv16, v_split_n;   // MN-major V descriptor fields (16-byte units)
 };
 
-template <int D, int KV>
+// BIAS of the kernel: none, the logarithmic distance bias, the distance table
+enum TcBias : int { kNoBias = 0, kLogBias = 1, kTableBias = 2 };
+static constexpr int kTabHeads = 16;                     // heads per CTA with a distance table (bounds its staging)
+
+template <int D, int KV, int BIAS>
 struct TcSmem {
+  // distance table: per KV tile the entries of its KV + tokens - 1 distances x GP heads, double buffered
+  static constexpr int kTabFloats = KV * kTabHeads + kTcRows;
+  static constexpr int kTabBytes = BIAS == kTableBias ? 2 * kTabFloats * 4 : 0;
   static constexpr int kQBytes = kTcRows * D * 2;
   static constexpr int kTileBytes = KV * D * 2;            // one K (or V) tile
   static constexpr int kStageBytes = 2 * kTileBytes;
   static constexpr int kPBytes = kTcRows * KV * 2;
-  static constexpr int kFixed = kQBytes + 2 * kPBytes;
+  static constexpr int kFixed = kQBytes + 2 * kPBytes + kTabBytes;
   // as many KV stages as fit next to Q and the two P buffers (227 KB per CTA), at most 4
   static constexpr int kFit = (232448 - 2048 - kFixed) / kStageBytes;
   static constexpr int kStages = kFit > 4 ? 4 : kFit;
+  static constexpr int kTabOff = kQBytes + 2 * kPBytes + kStages * kStageBytes;
   static constexpr int kBarOff = kFixed + kStages * kStageBytes;
   static constexpr int kBytes = kBarOff + 256 + 1024;
   static constexpr int kTmemCols = (2 * KV + D) <= 128 ? 128 : ((2 * KV + D) <= 256 ? 256 : 512);
@@ -101,11 +109,11 @@ __device__ __forceinline__ uint32_t a_tile_off(int row, int c) {
   return (c >> 3) * (kTcRows * 128) + row * 128 + (((c & 7) ^ (row & 7)) << 4);
 }
 
-template <int D, int KV, bool CAP, bool BIAS>
+template <int D, int KV, bool CAP, int BIAS>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v,
                        const TcAttnParams p) {
-  using SM = TcSmem<D, KV>;
+  using SM = TcSmem<D, KV, BIAS>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sq = smem;
@@ -264,10 +272,31 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
     const int lim = ctx_len + tok;                       // last visible key of this row
     const int low = p.window > 0 ? lim - p.window + 1 : 0;          // first visible key of this row
     float b1 = 0.f, b2 = 0.f;
-    if (BIAS) { b1 = p.ex.r1[head]; b2 = p.ex.r2[head]; }
+    if (BIAS == kLogBias) { b1 = p.ex.r1[head]; b2 = p.ex.r2[head]; }
+    // distance table: entry (tile buffer b, distance offset k, head) at [b][k * GP + head]; the offset of key `key` for
+    // this row is row / GP + KV - 1 - (key - key0), so the lanes of a warp read neighbouring words
+    float* stab = reinterpret_cast<float*>(smem + SM::kTabOff);
+    if (BIAS == kTableBias) b1 = dist_table_log2(p.ex.dtab + head, p.ex.dtab_n, p.Hq, p.ex.dtab_n - 1);
     float m_run = -INFINITY, l_run = 0.f;
     for (int tile = 0; tile < n_tiles; ++tile) {
       const int b = tile & 1;
+      bool far_tile = false;
+      const float* trow = stab;
+      if (BIAS == kTableBias) {
+        // smallest distance of the tile (CTA-uniform); at the table's end every score gets the same entry
+        const int d0 = ctx_len + tok_base - ((tile0 + tile) * KV + KV - 1);
+        far_tile = d0 >= p.ex.dtab_n - 1;
+        if (!far_tile) {
+          float* dst = stab + b * SM::kTabFloats;
+          for (int e = row; e < (KV - 1) * p.GP + kTcRows; e += kTcRows) {
+            const int k = e / p.GP;
+            dst[e] = dist_table_log2(p.ex.dtab + hbase + (e - k * p.GP), p.ex.dtab_n, p.Hq, d0 + k);
+          }
+          // one barrier per tile is enough: buffer b was last read two tiles ago, before the previous barrier
+          asm volatile("bar.sync 1, 128;" ::: "memory");
+          trow = dst + row;
+        }
+      }
       mbar_wait(&s_full[b], (tile >> 1) & 1);
       tc_fence_after();
       const uint32_t t_s = tmem + lane_base + b * KV;
@@ -282,11 +311,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
         uint32_t v[32];
         tmem_ld_32x32(t_s + c, v);
         tmem_ld_wait();
-        if (BIAS) {
+        if (BIAS == kLogBias) {
 #pragma unroll
           for (int e = 0; e < 32; ++e) {
             const int key = key0 + c + e;
             const float x = fmaf(__uint_as_float(v[e]), p.scale_log2, -dist_bias_log2(b1, b2, lim - key));
+            mx = fmaxf(mx, (key <= lim && key >= low) ? x : -INFINITY);
+          }
+        } else if (BIAS == kTableBias && !far_tile) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) {
+            const int key = key0 + c + e;
+            const float x = fmaf(__uint_as_float(v[e]), p.scale_log2, trow[(KV - 1 - c - e) * p.GP]);
             mx = fmaxf(mx, (key <= lim && key >= low) ? x : -INFINITY);
           }
         } else if (need_mask) {
@@ -299,7 +335,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
         }
       }
       // the cap is increasing in the score: the capped maximum is the cap of the raw maximum
-      const float mx_s = BIAS ? mx : !CAP ? mx * p.scale_log2
+      const float mx_s = BIAS == kLogBias || (BIAS == kTableBias && !far_tile) ? mx
+                         : BIAS == kTableBias ? fmaf(mx, p.scale_log2, b1)
+                         : !CAP ? mx * p.scale_log2
                               : (mx == -INFINITY ? -INFINITY : p.cap_log2 * tanh_exp(mx * p.scale_over_cap));
       const float m_new = fmaxf(m_run, mx_s);
       const float m_use = (m_new == -INFINITY) ? 0.f : m_new;
@@ -316,8 +354,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
         float f[32];
 #pragma unroll
         for (int e = 0; e < 32; ++e) {
-          float x = BIAS ? exp2f(fmaf(__uint_as_float(v[e]), p.scale_log2,
-                                      -dist_bias_log2(b1, b2, lim - (key0 + c + e)) - m_use))
+          float x = BIAS == kLogBias ? exp2f(fmaf(__uint_as_float(v[e]), p.scale_log2,
+                                                  -dist_bias_log2(b1, b2, lim - (key0 + c + e)) - m_use))
+                    : BIAS == kTableBias
+                        ? exp2f(fmaf(__uint_as_float(v[e]), p.scale_log2,
+                                     (far_tile ? b1 : trow[(KV - 1 - c - e) * p.GP]) - m_use))
                     : CAP ? exp2f(fmaf(p.cap_log2, tanh_exp(__uint_as_float(v[e]) * p.scale_over_cap), -m_use))
                         : exp2f(fmaf(__uint_as_float(v[e]), p.scale_log2, -m_use));
           if (need_mask && (key0 + c + e > lim || key0 + c + e < low)) x = 0.f;
@@ -473,10 +514,10 @@ static int get_kv_slab_tmap(const void* base, int64_t num_pages, int Hkv, int D,
   return 0;
 }
 
-template <int D, int KV, bool CAP = false, bool BIAS = false>
+template <int D, int KV, bool CAP = false, int BIAS = kNoBias>
 static int launch_prefill_tc(const CUtensorMap& tk, const CUtensorMap& tv, const TcAttnParams& p, int num_seqs,
                              int max_q_len, cudaStream_t st) {
-  using SM = TcSmem<D, KV>;
+  using SM = TcSmem<D, KV, BIAS>;
   static PerDeviceOnce configured;
   if (configured.need()) {
     CUDA_CHECK_RET(cudaFuncSetAttribute(attn_prefill_tc_kernel<D, KV, CAP, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -505,7 +546,8 @@ static int attn_prefill_tc_impl(const void* q, int64_t q_ts, void* out, const vo
                                 const AttnExtras& ex = AttnExtras()) {
   if (num_seqs <= 0 || max_q_len <= 0) return 0;
   if ((D != 64 && D != 128) || (kv_tile != 64 && kv_tile != 128) || page_size < 8 || kv_tile % page_size != 0 ||
-      Hq % Hkv != 0 || (ex.r1 != nullptr && softcap > 0.f))
+      Hq % Hkv != 0 || ((ex.r1 != nullptr || ex.dtab != nullptr) && softcap > 0.f) ||
+      (ex.dtab != nullptr && (ex.r1 != nullptr || kv_tile != 64)))
     return 2;
   CUtensorMap tk, tv;
   if (get_kv_slab_tmap(k_cache, num_pages, Hkv, D, page_size, &tk)) return 1;
@@ -519,7 +561,7 @@ static int attn_prefill_tc_impl(const void* q, int64_t q_ts, void* out, const vo
   p.max_blocks = max_blocks; p.Hq = Hq; p.Hkv = Hkv; p.G = Hq / Hkv;
   p.GP = 1;
   for (int d = (p.G < kTcRows ? p.G : kTcRows); d >= 1; --d)
-    if (p.G % d == 0 && kTcRows % d == 0) { p.GP = d; break; }
+    if (p.G % d == 0 && kTcRows % d == 0 && (ex.dtab == nullptr || d <= kTabHeads)) { p.GP = d; break; }
   p.page_size = page_size; p.seq_offset = seq_offset;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
@@ -540,13 +582,17 @@ static int attn_prefill_tc_impl(const void* q, int64_t q_ts, void* out, const vo
     }
   }
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (ex.dtab != nullptr) {
+    return D == 128 ? launch_prefill_tc<128, 64, false, kTableBias>(tk, tv, p, num_seqs, max_q_len, st)
+                    : launch_prefill_tc<64, 64, false, kTableBias>(tk, tv, p, num_seqs, max_q_len, st);
+  }
   if (ex.r1 != nullptr) {
     if (D == 128) {
-      return kv_tile == 128 ? launch_prefill_tc<128, 128, false, true>(tk, tv, p, num_seqs, max_q_len, st)
-                            : launch_prefill_tc<128, 64, false, true>(tk, tv, p, num_seqs, max_q_len, st);
+      return kv_tile == 128 ? launch_prefill_tc<128, 128, false, kLogBias>(tk, tv, p, num_seqs, max_q_len, st)
+                            : launch_prefill_tc<128, 64, false, kLogBias>(tk, tv, p, num_seqs, max_q_len, st);
     }
-    return kv_tile == 128 ? launch_prefill_tc<64, 128, false, true>(tk, tv, p, num_seqs, max_q_len, st)
-                          : launch_prefill_tc<64, 64, false, true>(tk, tv, p, num_seqs, max_q_len, st);
+    return kv_tile == 128 ? launch_prefill_tc<64, 128, false, kLogBias>(tk, tv, p, num_seqs, max_q_len, st)
+                          : launch_prefill_tc<64, 64, false, kLogBias>(tk, tv, p, num_seqs, max_q_len, st);
   }
   if (softcap > 0.f) {
     if (D == 128) {
@@ -583,8 +629,8 @@ GLLM_EXPORT int gllm_attn_prefill_tc_cap(const void* q, int64_t q_ts, void* out,
                                          int max_q_len, int max_blocks, int Hq, int Hkv, int D, int page_size,
                                          float scale, int kv_tile, const void* sink, float softcap, int window,
                                          int64_t out_ts, const void* r1, const void* r2, const void* gate, int64_t ldg,
-                                         const void* v_turn, void* stream) {
+                                         const void* v_turn, const void* dtab, int dtab_n, void* stream) {
   return attn_prefill_tc_impl(q, q_ts, out, k_cache, v_cache, num_pages, block_table, seq_lens, q_start, num_seqs,
                               seq_offset, max_q_len, max_blocks, Hq, Hkv, D, page_size, scale, kv_tile, sink, softcap,
-                              stream, window, out_ts, make_extras(r1, r2, gate, ldg, v_turn));
+                              stream, window, out_ts, make_extras(r1, r2, gate, ldg, v_turn, dtab, dtab_n));
 }

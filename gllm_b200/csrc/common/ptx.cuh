@@ -302,6 +302,12 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))), written as z sigmoid of twice the tanh's argument
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+  const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+  return __fdividef(z, 1.0f + __expf(fminf(-2.0f * u, 80.0f)));
+}
+
 __device__ __forceinline__ float2 unpack_bf16(uint32_t u) {
   __nv_bfloat162 v = *reinterpret_cast<__nv_bfloat162*>(&u);
   return __bfloat1622float2(v);

@@ -63,6 +63,7 @@ struct GemmParams {
   // gated epilogue variant (kEpiSiluMul with glu_limit > 0): g = min(gate, limit), u = clamp(up, +-limit),
   // out = g * sigmoid(glu_alpha * g) * (u + 1) instead of silu(gate) * up
   float glu_limit, glu_alpha;
+  int gelu;   // kEpiSiluMul: the tanh form of gelu instead of silu
   // plain-store epilogue activation: 0 none, 1 squared ReLU (max(x, 0)^2, after the bias)
   int act;
   // split-K (decode-sized M): unit = (tile, k-slice); partials go through an fp32 workspace in a
@@ -431,6 +432,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
                   const float gc = fminf(gv, p.glu_limit);
                   const float uc = fminf(fmaxf(uv, -p.glu_limit), p.glu_limit);
                   f[e] = gc / (1.0f + __expf(-p.glu_alpha * gc)) * (uc + 1.0f);
+                } else if (p.gelu) {
+                  f[e] = gelu_tanh_fast(gv) * uv;
                 } else {
                   f[e] = gv / (1.0f + __expf(-gv)) * uv;
                 }
@@ -622,7 +625,7 @@ GLLM_EXPORT int gllm_gemm_tune(int force_split, int max_split_m) {
 static int gemm_bf16_impl(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc, int M, int N,
                           int K, const void* bias, int epi, int force_bn, const GemmComm* comm, void* ws,
                           int64_t ws_bytes, void* tile_cnt, int max_tiles, void* stream, float glu_limit,
-                          float glu_alpha) {
+                          float glu_alpha, int gelu = 0) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if ((K % 8) != 0 || (N % 8) != 0 || (lda % 8) != 0 || (ldw % 8) != 0 || (ldc % 8) != 0) {
     fprintf(stderr, "[gllm_b200] gemm_bf16: K, N and leading dims must be multiples of 8\n");
@@ -644,6 +647,7 @@ static int gemm_bf16_impl(const void* A, int64_t lda, const void* W, int64_t ldw
   p.bias = reinterpret_cast<const __nv_bfloat16*>(bias);
   p.glu_limit = glu_limit;
   p.glu_alpha = glu_alpha;
+  p.gelu = gelu;
   if (comm != nullptr) {
     p.a_ready = comm->a_ready;
     p.a_expected = comm->a_expected;
@@ -692,6 +696,15 @@ GLLM_EXPORT int gllm_gemm_bf16_glu(const void* A, int64_t lda, const void* W, in
   if (limit <= 0.f) return 1;
   return gemm_bf16_impl(A, lda, W, ldw, C, ldc, M, N, K, nullptr, kEpiSiluMul, 256, nullptr, ws, ws_bytes, tile_cnt,
                         max_tiles, stream, limit, alpha);
+}
+
+// Gate / up projection with the tanh-gelu gated epilogue (weight rows interleaved per 128, BN = 256):
+// C[:, f] = gelu_tanh(gate) up.
+GLLM_EXPORT int gllm_gemm_bf16_gelu(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
+                                    int M, int N, int K, void* ws, int64_t ws_bytes, void* tile_cnt, int max_tiles,
+                                    void* stream) {
+  return gemm_bf16_impl(A, lda, W, ldw, C, ldc, M, N, K, nullptr, kEpiSiluMul, 256, nullptr, ws, ws_bytes, tile_cnt,
+                        max_tiles, stream, 0.f, 0.f, 1);
 }
 
 // Number of (m_tile, n_tile) pairs whose rows intersect [row0, row1) — used by the consumer

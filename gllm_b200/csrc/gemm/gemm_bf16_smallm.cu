@@ -34,7 +34,7 @@ struct SmallMParams {
   const __nv_bfloat16* bias;
   float* ws;              // [num_n_tiles * S][128][BT] fp32 partials
   uint32_t* counters;     // [num_n_tiles], zero on entry, self-resetting
-  int silu;               // 1: weight rows interleaved per 128: tile 2g = gate, tile 2g+1 = up
+  int silu;               // gated epilogue (1: silu, 2: the tanh form of gelu): weight rows interleaved per 128: tile 2g = gate, tile 2g+1 = up
   int stages;
   uint32_t tmem_cols;
 };
@@ -266,10 +266,11 @@ gemm_smallm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
             for (int uu = 0; uu < U; ++uu) {
               const int m = m0 + uu * 4 + mr;
               if (m < p.M && f + 3 < p.N / 2) {
-                const float o0 = g[uu].x / (1.f + __expf(-g[uu].x)) * up[uu].x;
-                const float o1 = g[uu].y / (1.f + __expf(-g[uu].y)) * up[uu].y;
-                const float o2 = g[uu].z / (1.f + __expf(-g[uu].z)) * up[uu].z;
-                const float o3 = g[uu].w / (1.f + __expf(-g[uu].w)) * up[uu].w;
+                auto act = [&](float z) { return p.silu == 2 ? gelu_tanh_fast(z) : z / (1.f + __expf(-z)); };
+                const float o0 = act(g[uu].x) * up[uu].x;
+                const float o1 = act(g[uu].y) * up[uu].y;
+                const float o2 = act(g[uu].z) * up[uu].z;
+                const float o3 = act(g[uu].w) * up[uu].w;
                 *reinterpret_cast<uint2*>(p.C + static_cast<size_t>(m) * p.ldc + f) =
                     make_uint2(pack_bf16(o0, o1), pack_bf16(o2, o3));
               }
@@ -294,7 +295,7 @@ gemm_smallm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
 using namespace b200;
 
 // ws: fp32 workspace of at least gllm_gemm_smallm_ws_floats() elements; counters: >= ceil(N/128)
-// uint32 zeros. silu: weight rows interleaved per 128 (gate|up), output has N/2 columns.
+// uint32 zeros. silu: weight rows interleaved per 128 (gate|up), output has N/2 columns (1: silu, 2: tanh gelu).
 GLLM_EXPORT int gllm_gemm_smallm(const void* A, int64_t lda, const void* W, int64_t ldw, void* C, int64_t ldc,
                                  int M, int N, int K, const void* bias, int silu, int force_split, void* ws,
                                  int64_t ws_floats, void* counters, void* stream) {

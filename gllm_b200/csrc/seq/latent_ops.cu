@@ -199,13 +199,20 @@ __global__ void __launch_bounds__(128) latent_norm_rope_write_kernel(
     const T* __restrict__ q, long ldq_t, long ldq_h, int H, int dim, const T* __restrict__ dkv, long ldkv, int rank,
     int rot, const T* __restrict__ norm_w, float eps, const int* __restrict__ positions,
     const float* __restrict__ freqs, float mag, T* __restrict__ q_full, T* __restrict__ cache,
-    const int* __restrict__ slots, int ps, int slab) {
+    const int* __restrict__ slots, int ps, int slab, const float* __restrict__ angles) {
   extern __shared__ float cs[];          // [rot / 2][2]: cos, sin
   __shared__ float scratch[4];
   const int t = blockIdx.x;
   const int half = rot / 2;
   const float pos = (float)positions[t];
+  // entries of pair i: neighbours, or (angles given) half the rotated part apart
+  const int ma = angles != nullptr ? 1 : 2, ob = angles != nullptr ? half : 1;
   for (int i = threadIdx.x; i < half; i += 128) {
+    if (angles != nullptr) {
+      cs[2 * i] = angles[(size_t)t * rot + i];
+      cs[2 * i + 1] = angles[(size_t)t * rot + half + i];
+      continue;
+    }
     const float ang = pos * freqs[i];
     cs[2 * i] = cosf(ang) * mag;
     cs[2 * i + 1] = sinf(ang) * mag;
@@ -221,31 +228,32 @@ __global__ void __launch_bounds__(128) latent_norm_rope_write_kernel(
     for (int d = threadIdx.x; d < rank; d += 128)
       cache[cache_index(slot, 0, d, 1, Dl, ps, slab)] = from_f<T>(to_f(row[d]) * r * to_f(norm_w[d]));
     for (int i = threadIdx.x; i < half; i += 128) {
-      const float a = to_f(row[rank + 2 * i]), b = to_f(row[rank + 2 * i + 1]);
+      const float a = to_f(row[rank + ma * i]), b = to_f(row[rank + ma * i + ob]);
       const float c = cs[2 * i], s = cs[2 * i + 1];
-      cache[cache_index(slot, 0, rank + 2 * i, 1, Dl, ps, slab)] = from_f<T>(a * c - b * s);
-      cache[cache_index(slot, 0, rank + 2 * i + 1, 1, Dl, ps, slab)] = from_f<T>(b * c + a * s);
+      cache[cache_index(slot, 0, rank + ma * i, 1, Dl, ps, slab)] = from_f<T>(a * c - b * s);
+      cache[cache_index(slot, 0, rank + ma * i + ob, 1, Dl, ps, slab)] = from_f<T>(b * c + a * s);
     }
   }
   for (int idx = threadIdx.x; idx < H * half; idx += 128) {
     const int h = idx / half, i = idx - h * half;
     const T* qr = q + (size_t)t * ldq_t + (size_t)h * ldq_h + dim;
-    const float a = to_f(qr[2 * i]), b = to_f(qr[2 * i + 1]);
+    const float a = to_f(qr[ma * i]), b = to_f(qr[ma * i + ob]);
     const float c = cs[2 * i], s = cs[2 * i + 1];
     T* dst = q_full + ((size_t)t * H + h) * Dl + rank;
-    dst[2 * i] = from_f<T>(a * c - b * s);
-    dst[2 * i + 1] = from_f<T>(b * c + a * s);
+    dst[ma * i] = from_f<T>(a * c - b * s);
+    dst[ma * i + ob] = from_f<T>(b * c + a * s);
   }
 }
 
 // Plain causal multi-query attention over the latent cache: one warp per (token, head), 4 consecutive tokens of one
 // head per block. Keys are the rows [latent | rotated key] of width Dl, values their first `rank` columns. Scores:
-// one key per lane; P.V: value columns across lanes.
+// one key per lane; P.V: value columns across lanes. window > 0: position i sees j with i - j < window; sink (per head,
+// optional): one more logit in the denominator that carries no value.
 template <typename T, int MAXR>
 __global__ void __launch_bounds__(128) latent_attn_kernel(
     const T* __restrict__ q, const T* __restrict__ cache, const int* __restrict__ block_table, int bt_stride,
     const int* __restrict__ qsl, const int* __restrict__ positions, int ntok, int nseq, float scale, int H, int Dl,
-    int rank, T* __restrict__ out, int ps, int slab) {
+    int rank, T* __restrict__ out, int ps, int slab, int window, const float* __restrict__ sink) {
   extern __shared__ float qs_all[];      // [4][Dl]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + warp, h = blockIdx.y;
@@ -259,11 +267,11 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(
   const int* bt = block_table + (size_t)s * bt_stride;
   const int nslab = Dl / slab;
   const size_t page_stride = (size_t)Dl * ps;
-  float m = -INFINITY, l = 0.f;
+  float m = sink != nullptr ? sink[h] : -INFINITY, l = sink != nullptr ? 1.0f : 0.0f;
   float acc[MAXR];
 #pragma unroll
   for (int r = 0; r < MAXR; ++r) acc[r] = 0.f;
-  for (int j0 = 0; j0 <= i; j0 += 32) {
+  for (int j0 = window > 0 ? max(0, i - window + 1) : 0; j0 <= i; j0 += 32) {
     const int j = j0 + lane;
     const bool valid = j <= i;
     size_t base = 0;
@@ -422,6 +430,31 @@ __global__ void __launch_bounds__(128) grouped_router_select_kernel(
 }
 
 // out[t, f] = g sigmoid(alpha g) (u + 1), g = min(gu[t, f], limit), u = clamp(gu[t, F + f], +-limit)
+// o[t, i] *= sigmoid(gate[t, i]), in place; bf16 rows in 16-byte pieces (VEC 8) or single entries (VEC 1)
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) gate_rows_kernel(T* __restrict__ o, long ldo, const T* __restrict__ gate, long ldg,
+                                                        int pieces, size_t total) {
+  const size_t i = (size_t)blockIdx.x * 256 + threadIdx.x;
+  if (i >= total) return;
+  const size_t t = i / pieces, c = (i - t * pieces) * VEC;
+  T* op = o + t * ldo + c;
+  const T* gp = gate + t * ldg + c;
+  if constexpr (VEC == 8) {
+    uint4 a = *reinterpret_cast<const uint4*>(op);
+    const uint4 b = *reinterpret_cast<const uint4*>(gp);
+    __nv_bfloat162* x = reinterpret_cast<__nv_bfloat162*>(&a);
+    const __nv_bfloat162* g = reinterpret_cast<const __nv_bfloat162*>(&b);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 v = __bfloat1622float2(x[e]), z = __bfloat1622float2(g[e]);
+      x[e] = __floats2bfloat162_rn(v.x * sigmoid_f(z.x), v.y * sigmoid_f(z.y));
+    }
+    *reinterpret_cast<uint4*>(op) = a;
+  } else {
+    op[0] = from_f<T>(to_f(op[0]) * sigmoid_f(to_f(gp[0])));
+  }
+}
+
 template <typename T>
 __global__ void glu_clamp_kernel(const T* __restrict__ gu, long ld, int F, T* __restrict__ out, size_t total,
                                  float limit, float alpha) {
@@ -539,7 +572,7 @@ GLLM_EXPORT int gllm_lat_norm_rope_write(const void* q, long ldq_t, long ldq_h, 
                                          long ldkv, int rank, int rot, const void* norm_w, float eps,
                                          const void* positions, const void* freqs, float mag, void* q_full,
                                          void* cache, const void* slots, int ps, int slab, int ntok, int is_f32,
-                                         void* stream) {
+                                         const void* angles, void* stream) {
   if (ntok <= 0) return 0;
   if (rot % 2 != 0) return 2;
   cudaStream_t st = (cudaStream_t)stream;
@@ -548,11 +581,11 @@ GLLM_EXPORT int gllm_lat_norm_rope_write(const void* q, long ldq_t, long ldq_h, 
                 (latent_norm_rope_write_kernel<bf16_t><<<ntok, 128, smem, st>>>(
                     (const bf16_t*)q, ldq_t, ldq_h, H, dim, (const bf16_t*)dkv, ldkv, rank, rot, (const bf16_t*)norm_w,
                     eps, (const int*)positions, (const float*)freqs, mag, (bf16_t*)q_full, (bf16_t*)cache,
-                    (const int*)slots, ps, slab)),
+                    (const int*)slots, ps, slab, (const float*)angles)),
                 (latent_norm_rope_write_kernel<float><<<ntok, 128, smem, st>>>(
                     (const float*)q, ldq_t, ldq_h, H, dim, (const float*)dkv, ldkv, rank, rot, (const float*)norm_w,
                     eps, (const int*)positions, (const float*)freqs, mag, (float*)q_full, (float*)cache,
-                    (const int*)slots, ps, slab)));
+                    (const int*)slots, ps, slab, (const float*)angles)));
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
 }
@@ -561,13 +594,14 @@ namespace {
 template <typename T>
 int latent_attn_dispatch(dim3 grid, size_t smem, cudaStream_t st, const void* q, const void* cache, const int* bt,
                          int bt_stride, const int* qsl, const int* pos, int ntok, int nseq, float scale, int H, int Dl,
-                         int rank, void* out, int ps, int slab) {
+                         int rank, void* out, int ps, int slab, int window, const float* sink) {
 #define GLLM_LATTN(R)                                                                                          \
   do {                                                                                                         \
     if (smem > 48 * 1024)                                                                                      \
       cudaFuncSetAttribute(latent_attn_kernel<T, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);  \
     latent_attn_kernel<T, R><<<grid, 128, smem, st>>>((const T*)q, (const T*)cache, bt, bt_stride, qsl, pos,    \
-                                                      ntok, nseq, scale, H, Dl, rank, (T*)out, ps, slab);       \
+                                                      ntok, nseq, scale, H, Dl, rank, (T*)out, ps, slab,        \
+                                                      window, sink);                                           \
   } while (0)
   if (rank <= 64) GLLM_LATTN(2);
   else if (rank <= 128) GLLM_LATTN(4);
@@ -581,7 +615,8 @@ int latent_attn_dispatch(dim3 grid, size_t smem, cudaStream_t st, const void* q,
 
 GLLM_EXPORT int gllm_lat_attention(const void* q, const void* cache, const void* block_table, int bt_stride,
                                    const void* qsl, const void* positions, int ntok, int nseq, float scale, int H,
-                                   int Dl, int rank, void* out, int ps, int slab, int is_f32, void* stream) {
+                                   int Dl, int rank, void* out, int ps, int slab, int is_f32, int window,
+                                   const void* sink, void* stream) {
   if (ntok <= 0) return 0;
   if (Dl % slab != 0 || rank > Dl) return 2;
   cudaStream_t st = (cudaStream_t)stream;
@@ -591,10 +626,12 @@ GLLM_EXPORT int gllm_lat_attention(const void* q, const void* cache, const void*
   int rc;
   if (is_f32)
     rc = latent_attn_dispatch<float>(grid, smem, st, q, cache, (const int*)block_table, bt_stride, (const int*)qsl,
-                                     (const int*)positions, ntok, nseq, scale, H, Dl, rank, out, ps, slab);
+                                     (const int*)positions, ntok, nseq, scale, H, Dl, rank, out, ps, slab, window,
+                                     (const float*)sink);
   else
     rc = latent_attn_dispatch<bf16_t>(grid, smem, st, q, cache, (const int*)block_table, bt_stride, (const int*)qsl,
-                                      (const int*)positions, ntok, nseq, scale, H, Dl, rank, out, ps, slab);
+                                      (const int*)positions, ntok, nseq, scale, H, Dl, rank, out, ps, slab, window,
+                                      (const float*)sink);
   if (rc) return rc;
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
@@ -612,6 +649,26 @@ GLLM_EXPORT int gllm_lat_grouped_router_select(const void* logits, const void* c
   grouped_router_select_kernel<<<(ntok + 3) / 4, 128, smem, st>>>((const float*)logits, (const float*)correction,
                                                                   ntok, E, top_k, n_groups, keep, scale,
                                                                   (float*)wout, (int*)ids, sigmoid, group_top, renorm);
+  CUDA_CHECK_RET(cudaGetLastError());
+  return 0;
+}
+
+GLLM_EXPORT int gllm_lat_gate_rows(void* o, long ldo, const void* gate, long ldg, int ntok, int n, int is_f32,
+                                   void* stream) {
+  if (ntok <= 0 || n <= 0) return 0;
+  cudaStream_t st = (cudaStream_t)stream;
+  if (!is_f32 && n % 8 == 0 && ldo % 8 == 0 && ldg % 8 == 0 && (((uintptr_t)o | (uintptr_t)gate) & 15) == 0) {
+    const size_t total = (size_t)ntok * (n / 8);
+    gate_rows_kernel<bf16_t, 8><<<(unsigned)((total + 255) / 256), 256, 0, st>>>((bf16_t*)o, ldo, (const bf16_t*)gate, ldg,
+                                                                               n / 8, total);
+    CUDA_CHECK_RET(cudaGetLastError());
+    return 0;
+  }
+  const size_t total = (size_t)ntok * n;
+  const unsigned blocks = (unsigned)((total + 255) / 256);
+  GLLM_BY_DTYPE(is_f32,
+                (gate_rows_kernel<bf16_t, 1><<<blocks, 256, 0, st>>>((bf16_t*)o, ldo, (const bf16_t*)gate, ldg, n, total)),
+                (gate_rows_kernel<float, 1><<<blocks, 256, 0, st>>>((float*)o, ldo, (const float*)gate, ldg, n, total)));
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
 }

@@ -34,14 +34,15 @@ __global__ void embed_scale_kernel(const int* __restrict__ ids, const T* __restr
 // layer scale). With emit_plain and no w_pre, out = x rounded to T (sublayers that read the stream un-normed).
 // w_off is added to both norm weights in fp32 (1 for weights stored around zero); out_mul multiplies the normed
 // output (a logit scale applied to the final norm's result, before it is rounded). y_mul multiplies the branch (a
-// residual multiplier); without w_post the branch is added as it is: x += y_mul * y.
+// residual multiplier); without w_post the branch is added as it is: x += y_mul * y. center: the pre-norm is a layer norm without
+// a bias, (x - mean) / sqrt(mean of the squared deviations + eps) * w_pre.
 template <typename T>
 __global__ void __launch_bounds__(256) resid_norm_kernel(float* __restrict__ x, const T* __restrict__ y, long ldy,
                                                          const T* __restrict__ w_post,
                                                          const float* __restrict__ post_scale,
                                                          const float* __restrict__ add, const T* __restrict__ w_pre,
                                                          T* __restrict__ out, int width, float eps, int emit_plain,
-                                                         float w_off, float out_mul, float y_mul) {
+                                                         float w_off, float out_mul, float y_mul, int center) {
   __shared__ float scratch[8];
   const int t = blockIdx.x;
   float* xr = x + (size_t)t * width;
@@ -67,13 +68,20 @@ __global__ void __launch_bounds__(256) resid_norm_kernel(float* __restrict__ x, 
     if (add != nullptr) v += add[(size_t)t * width + i];
     if (y != nullptr || add != nullptr) xr[i] = v;
     if (plain) out[(size_t)t * width + i] = from_f<T>(v);
-    ss2 += v * v;
+    ss2 += center ? v : v * v;
   }
   if (w_pre == nullptr) return;
   ss2 = block_sum<256>(ss2, scratch);
+  float mean = 0.f;
+  if (center) {                          // the sum was that of the values; now the squared deviations
+    mean = ss2 / (float)width;
+    ss2 = 0.f;
+    for (int i = threadIdx.x; i < width; i += 256) { const float d = xr[i] - mean; ss2 += d * d; }
+    ss2 = block_sum<256>(ss2, scratch);
+  }
   const float r = 1.0f / sqrtf(ss2 / (float)width + eps);
   for (int i = threadIdx.x; i < width; i += 256)
-    out[(size_t)t * width + i] = from_f<T>(xr[i] * r * (to_f(w_pre[i]) + w_off) * out_mul);
+    out[(size_t)t * width + i] = from_f<T>((xr[i] - mean) * r * (to_f(w_pre[i]) + w_off) * out_mul);
 }
 
 
@@ -83,7 +91,8 @@ template <int MAXP>
 __global__ void __launch_bounds__(256) resid_norm_vec_kernel(
     float* __restrict__ x, const __nv_bfloat16* __restrict__ y, long ldy, const __nv_bfloat16* __restrict__ w_post,
     const float* __restrict__ post_scale, const float* __restrict__ add, const __nv_bfloat16* __restrict__ w_pre,
-    __nv_bfloat16* __restrict__ out, int width, float eps, int emit_plain, float w_off, float out_mul, float y_mul) {
+    __nv_bfloat16* __restrict__ out, int width, float eps, int emit_plain, float w_off, float out_mul, float y_mul,
+    int center) {
   __shared__ float scratch[8];
   const size_t row = (size_t)blockIdx.x * width;
   auto load8 = [](const __nv_bfloat16* ptr, float (&f)[8]) {
@@ -158,11 +167,23 @@ __global__ void __launch_bounds__(256) resid_norm_vec_kernel(
       }
       if (plain) store8(out + row + i, v[k]);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) ss2 += v[k][e] * v[k][e];
+      for (int e = 0; e < 8; ++e) ss2 += center ? v[k][e] : v[k][e] * v[k][e];
     }
   }
   if (w_pre == nullptr) return;
   ss2 = block_sum<256>(ss2, scratch);
+  if (center) {                          // the sum was that of the values; now the squared deviations
+    const float mean = ss2 / (float)width;
+    ss2 = 0.f;
+#pragma unroll
+    for (int k = 0; k < MAXP; ++k) {
+      if ((threadIdx.x + k * 256) * 8 < width) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) { v[k][e] -= mean; ss2 += v[k][e] * v[k][e]; }
+      }
+    }
+    ss2 = block_sum<256>(ss2, scratch);
+  }
   const float r = 1.0f / sqrtf(ss2 / (float)width + eps);
 #pragma unroll
   for (int k = 0; k < MAXP; ++k) {
@@ -214,7 +235,7 @@ __global__ void qk_norm_kv_write_kernel(const T* __restrict__ qk, long ldqk, int
 // 4 consecutive tokens of one head per block (their key ranges overlap, so K/V rows are shared through L1).
 // Scores: one key per lane; P.V: value entries across lanes. softcap > 0: a scaled score s becomes
 // softcap * tanh(s / softcap) before the softmax. r1, r2 (per head, both or none): r1 ln(1 + r2 (i - j)) is taken off the
-// score of key j. v_turn [ntok, Dv] (cos | sin of the query's position per pair): the values are rotated, the result
+// score of key j. dtab [dtab_n, H]: row min(i - j, dtab_n - 1) is added to it. v_turn [ntok, Dv] (cos | sin of the query's position per pair): the values are rotated, the result
 // is turned back, entry m with m + Dv / 2. gate (row stride ldg): the result is multiplied by sigmoid(gate).
 template <typename T, int MAXR>
 __global__ void __launch_bounds__(128) window_attn_kernel(
@@ -222,7 +243,8 @@ __global__ void __launch_bounds__(128) window_attn_kernel(
     int bt_stride, const int* __restrict__ qsl, const int* __restrict__ positions, int ntok, int nseq, float scale,
     int H, int G, int D, int Dv, int window, int chunk, const float* __restrict__ sink, T* __restrict__ out, long ldo,
     float out_scale, int ps, int slab, int slab_v, float softcap, const float* __restrict__ r1,
-    const float* __restrict__ r2, const T* __restrict__ gate, long ldg, const float* __restrict__ v_turn) {
+    const float* __restrict__ r2, const T* __restrict__ gate, long ldg, const float* __restrict__ v_turn,
+    const float* __restrict__ dtab, int dtab_n) {
   __shared__ float qs[4][256];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + warp, h = blockIdx.y;
@@ -262,6 +284,7 @@ __global__ void __launch_bounds__(128) window_attn_kernel(
       sc = dot * scale;
       if (softcap > 0.f) sc = softcap * tanhf(sc / softcap);
       if (r1 != nullptr) sc -= r1[h] * log1pf(r2[h] * (float)(i - j));
+      if (dtab != nullptr) sc += dtab[(size_t)min(i - j, dtab_n - 1) * H + h];
     }
     const float m_new = fmaxf(m, warp_max(sc));
     const float alpha = expf(m - m_new);          // m == -inf only before the first key: exp(-inf) == 0
@@ -588,12 +611,12 @@ int attn_dispatch(dim3 grid, cudaStream_t st, const void* q, const void* kc, con
                   int bt_stride, const int* qsl, const int* pos, int ntok, int nseq, float scale, int H, int G, int D,
                   int Dv, int window, int chunk, const float* sink, void* out, long ldo, float out_scale, int ps,
                   int slab, int slab_v, float softcap, const float* r1, const float* r2, const void* gate, long ldg,
-                  const float* v_turn) {
+                  const float* v_turn, const float* dtab, int dtab_n) {
 #define GLLM_ATTN(R)                                                                                              \
   window_attn_kernel<T, R><<<grid, 128, 0, st>>>((const T*)q, (const T*)kc, (const T*)vc, bt, bt_stride, qsl, pos, \
                                                  ntok, nseq, scale, H, G, D, Dv, window, chunk, sink, (T*)out, ldo, \
                                                  out_scale, ps, slab, slab_v, softcap, r1, r2, (const T*)gate, ldg, \
-                                                 v_turn)
+                                                 v_turn, dtab, dtab_n)
   if (D > 256) return 2;
   if (Dv <= 32) GLLM_ATTN(1);
   else if (Dv <= 64) GLLM_ATTN(2);
@@ -624,7 +647,7 @@ GLLM_EXPORT int gllm_seq_embed_scale(const void* ids, const void* table, void* o
 
 GLLM_EXPORT int gllm_seq_resid_norm(void* x, const void* y, long ldy, const void* w_post, const void* post_scale,
                                     const void* add, const void* w_pre, void* out, int ntok, int width, float eps,
-                                    int emit_plain, int is_f32, float w_off, float out_mul, float y_mul,
+                                    int emit_plain, int is_f32, float w_off, float out_mul, float y_mul, int center,
                                     void* stream) {
   if (ntok <= 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
@@ -635,7 +658,8 @@ GLLM_EXPORT int gllm_seq_resid_norm(void* x, const void* y, long ldy, const void
   resid_norm_vec_kernel<MP><<<ntok, 256, 0, st>>>((float*)x, (const __nv_bfloat16*)y, ldy,                          \
                                                   (const __nv_bfloat16*)w_post, (const float*)post_scale,           \
                                                   (const float*)add, (const __nv_bfloat16*)w_pre,                   \
-                                                  (__nv_bfloat16*)out, width, eps, emit_plain, w_off, out_mul, y_mul)
+                                                  (__nv_bfloat16*)out, width, eps, emit_plain, w_off, out_mul, y_mul, \
+                                                  center)
     if (width <= 2048) GLLM_RESID(1);
     else if (width <= 4096) GLLM_RESID(2);
     else GLLM_RESID(4);
@@ -647,11 +671,11 @@ GLLM_EXPORT int gllm_seq_resid_norm(void* x, const void* y, long ldy, const void
                 (resid_norm_kernel<__nv_bfloat16><<<ntok, 256, 0, st>>>(
                     (float*)x, (const __nv_bfloat16*)y, ldy, (const __nv_bfloat16*)w_post, (const float*)post_scale,
                     (const float*)add, (const __nv_bfloat16*)w_pre, (__nv_bfloat16*)out, width, eps, emit_plain,
-                    w_off, out_mul, y_mul)),
+                    w_off, out_mul, y_mul, center)),
                 (resid_norm_kernel<float><<<ntok, 256, 0, st>>>((float*)x, (const float*)y, ldy, (const float*)w_post,
                                                                 (const float*)post_scale, (const float*)add,
                                                                 (const float*)w_pre, (float*)out, width, eps,
-                                                                emit_plain, w_off, out_mul, y_mul)));
+                                                                emit_plain, w_off, out_mul, y_mul, center)));
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
 }
@@ -678,7 +702,8 @@ GLLM_EXPORT int gllm_seq_window_attention(const void* q, const void* kc, const v
                                           float scale, int H, int G, int D, int Dv, int window, int chunk,
                                           const void* sink, void* out, long ldo, float out_scale, int ps, int slab,
                                           int slab_v, int is_f32, float softcap, const void* r1, const void* r2,
-                                          const void* gate, long ldg, const void* v_turn, void* stream) {
+                                          const void* gate, long ldg, const void* v_turn, const void* dtab,
+                                          int dtab_n, void* stream) {
   if (ntok <= 0) return 0;
   if (v_turn != nullptr && Dv % 2 != 0) return 2;
   cudaStream_t st = (cudaStream_t)stream;
@@ -688,12 +713,13 @@ GLLM_EXPORT int gllm_seq_window_attention(const void* q, const void* kc, const v
     rc = attn_dispatch<float>(grid, st, q, kc, vc, (const int*)block_table, bt_stride, (const int*)qsl,
                               (const int*)positions, ntok, nseq, scale, H, G, D, Dv, window, chunk, (const float*)sink,
                               out, ldo, out_scale, ps, slab, slab_v, softcap, (const float*)r1, (const float*)r2, gate,
-                              ldg, (const float*)v_turn);
+                              ldg, (const float*)v_turn, (const float*)dtab, dtab_n);
   else
     rc = attn_dispatch<__nv_bfloat16>(grid, st, q, kc, vc, (const int*)block_table, bt_stride, (const int*)qsl,
                                       (const int*)positions, ntok, nseq, scale, H, G, D, Dv, window, chunk,
                                       (const float*)sink, out, ldo, out_scale, ps, slab, slab_v, softcap,
-                                      (const float*)r1, (const float*)r2, gate, ldg, (const float*)v_turn);
+                                      (const float*)r1, (const float*)r2, gate, ldg, (const float*)v_turn,
+                                      (const float*)dtab, dtab_n);
   if (rc) return rc;
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;

@@ -42,6 +42,32 @@ __global__ void __launch_bounds__(256) postnorm_kernel(float* __restrict__ x, co
   }
 }
 
+// Options of the rotary write below
+struct RowOptions {
+  int whole = 0;                 // the RMS norms run over all rows of q (of k) at once; weights [H * D] ([G * D])
+  float t_coef = 0.f;            // q times 1 + t_coef ln(floor((p + 1) / t_every) + 1) at position p (t_every > 0)
+  int t_every = 0;
+  const void* v_first = nullptr; // cached values: (1 - lam) v + lam v_first, rows ld_first elements apart
+  long ld_first = 0;
+  const float* lam = nullptr;    // one number
+};
+
+__device__ __forceinline__ float q_temperature(const RowOptions& ro, int pos) {
+  return ro.t_every > 0 ? fmaf(ro.t_coef, logf((float)((pos + 1) / ro.t_every + 1)), 1.0f) : 1.0f;
+}
+
+// 1 / root mean square of the H * D query entries and of the G * D key entries of one projected row (whole block)
+template <typename T>
+__device__ __forceinline__ float2 whole_row_scales(const T* __restrict__ row, int nq, int nk, float eps) {
+  __shared__ float scratch[2][8];
+  float sq = 0.f, sk = 0.f;
+  for (int i = threadIdx.x; i < nq; i += 256) { const float v = to_f(row[i]); sq += v * v; }
+  for (int i = threadIdx.x; i < nk; i += 256) { const float v = to_f(row[nq + i]); sk += v * v; }
+  sq = block_sum<256>(sq, scratch[0]);
+  sk = block_sum<256>(sk, scratch[1]);
+  return make_float2(1.0f / sqrtf(sq / (float)nq + eps), 1.0f / sqrtf(sk / (float)nk + eps));
+}
+
 // One block per token; its warps walk the heads: [0, H) queries, [H, H + G) keys, [H + G, H + 2G) values (copied to
 // the V cache). q / k: RMS norm over D with a shared weight, then entries i and i + rot/2 (i < rot/2) turn by
 // pos * base^(-2i/rot). The token's cos / sin row is formed once per block, the angle in fp64 (no table, no maximum
@@ -49,14 +75,15 @@ __global__ void __launch_bounds__(256) postnorm_kernel(float* __restrict__ x, co
 // frequencies); cos and sin are multiplied by `mag`. With G == 0 a row holds queries only (the keys and values are
 // another layer's) and no cache is touched. `unit`: q / k are divided by their root mean square without a weight.
 // `angles` [ntok, rot] (cos | sin, fp32): the row's table as formed once per step, used instead of positions and
-// frequencies; `v_angles` [ntok, Dv]: the values turn too, entry m with m + Dv / 2, and are cached so.
+// frequencies; `v_angles` [ntok, Dv]: the values turn too, entry m with m + Dv / 2, and are cached so. `ro` (RowOptions):
+// norms over the whole projection, query temperature, values mixed with another layer's.
 template <typename T>
 __global__ void __launch_bounds__(256) qk_norm_rope_kv_write_kernel(
     const T* __restrict__ qkv, long ld, int H, int G, int D, int Dv, const T* __restrict__ qn,
     const T* __restrict__ kn, float eps, const int* __restrict__ positions, int rot, double log2_base,
     T* __restrict__ q_out, T* __restrict__ kc, T* __restrict__ vc, const int* __restrict__ slots, int ps, int slab,
     int slab_v, const double* __restrict__ freqs, float mag, int unit, const float* __restrict__ angles,
-    const float* __restrict__ v_angles) {
+    const float* __restrict__ v_angles, const RowOptions ro) {
   extern __shared__ float cs_tab[];      // [rot / 2] cos, then [rot / 2] sin
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x;
@@ -73,6 +100,8 @@ __global__ void __launch_bounds__(256) qk_norm_rope_kv_write_kernel(
     cs_tab[i] = (float)(cs * (double)mag);
     cs_tab[half + i] = (float)(sn * (double)mag);
   }
+  const float2 rw = ro.whole ? whole_row_scales<T>(qkv + (size_t)t * ld, H * D, G * D, eps) : make_float2(1.f, 1.f);
+  const float temp = q_temperature(ro, positions[t]);
   __syncthreads();
   const int slot = G > 0 ? slots[t] : -1;
   for (int head = warp; head < H + 2 * G; head += 8) {
@@ -87,17 +116,29 @@ __global__ void __launch_bounds__(256) qk_norm_rope_kv_write_kernel(
         if (va != nullptr)
           o = from_f<T>(d < vh ? to_f(o) * va[d] - to_f(src[d + vh]) * va[vh + d]
                                : to_f(o) * va[d - vh] + to_f(src[d - vh]) * va[d]);
+        if (ro.v_first != nullptr) {
+          const float lam = *ro.lam;
+          const float f = to_f(reinterpret_cast<const T*>(ro.v_first)[(size_t)t * ro.ld_first + (size_t)g * Dv + d]);
+          o = from_f<T>((1.0f - lam) * to_f(o) + lam * f);
+        }
         vc[cache_index(slot, g, d, G, Dv, ps, slab_v)] = o;
       }
       continue;
     }
     if (head >= H && slot < 0) continue;
     const T* src = qkv + (size_t)t * ld + (size_t)head * D;
-    float ss = 0.f;
-    for (int d = lane; d < D; d += 32) { const float v = to_f(src[d]); ss += v * v; }
-    ss = warp_sum(ss);
     const T* w = head < H ? qn : kn;
-    const float r = w != nullptr || unit ? 1.0f / sqrtf(ss / (float)D + eps) : 1.0f;
+    float r;
+    if (ro.whole) {
+      r = head < H ? rw.x : rw.y;
+      w += (size_t)(head < H ? head : head - H) * D;
+    } else {
+      float ss = 0.f;
+      for (int d = lane; d < D; d += 32) { const float v = to_f(src[d]); ss += v * v; }
+      ss = warp_sum(ss);
+      r = w != nullptr || unit ? 1.0f / sqrtf(ss / (float)D + eps) : 1.0f;
+    }
+    if (head < H) r *= temp;
     for (int d = lane; d < D; d += 32) {
       float v = to_f(src[d]) * r * (w != nullptr ? to_f(w[d]) : 1.0f);
       if (d < rot) {
@@ -119,11 +160,29 @@ __global__ void __launch_bounds__(256) rope_kv_write_vec_kernel(
     const __nv_bfloat16* __restrict__ qkv, long ld, int H, int G, int D, int Dv, const __nv_bfloat16* __restrict__ qn,
     const __nv_bfloat16* __restrict__ kn, float eps, __nv_bfloat16* __restrict__ q_out, __nv_bfloat16* __restrict__ kc,
     __nv_bfloat16* __restrict__ vc, const int* __restrict__ slots, int ps, int slab, int slab_v, float mag, int unit,
-    const float* __restrict__ angles, const float* __restrict__ v_angles, int lanes) {
+    const float* __restrict__ angles, const float* __restrict__ v_angles, int lanes, const int* __restrict__ positions,
+    const RowOptions ro) {
   const int t = blockIdx.x;
   const int l = threadIdx.x % lanes, per = 256 / lanes;
   const int slot = slots[t];
   const int total = H + 2 * G, rounds = (total + per - 1) / per;
+  float2 rw = make_float2(1.f, 1.f);
+  if (ro.whole) {                                // 8-byte pieces, like everything here (H * D and G * D are multiples of 8)
+    __shared__ float scratch[2][8];
+    const __nv_bfloat16* row = qkv + (size_t)t * ld;
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x * 4; i < (H + G) * D; i += 1024) {
+      const uint2 a = *reinterpret_cast<const uint2*>(row + i);
+      const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.x));
+      const float2 y = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.y));
+      const float s = x.x * x.x + x.y * x.y + (y.x * y.x + y.y * y.y);
+      if (i < H * D) sq += s; else sk += s;
+    }
+    sq = block_sum<256>(sq, scratch[0]);
+    sk = block_sum<256>(sk, scratch[1]);
+    rw = make_float2(1.0f / sqrtf(sq / (float)(H * D) + eps), 1.0f / sqrtf(sk / (float)(G * D) + eps));
+  }
+  const float temp = q_temperature(ro, positions[t]);
   for (int r = 0; r < rounds; ++r) {             // every lane takes every round: the shuffles below need whole warps
     const int head = r * per + threadIdx.x / lanes;
     const bool is_v = head >= H + G, on = head < total && (head < H || slot >= 0);
@@ -148,11 +207,27 @@ __global__ void __launch_bounds__(256) rope_kv_write_vec_kernel(
     if (!mine) continue;
     const __nv_bfloat16* w = head < H ? qn : kn;
     if (!is_v && (w != nullptr || unit)) {
-      const float rn = 1.0f / sqrtf(ss / (float)D + eps);
+      float rn = head < H ? rw.x : rw.y;
+      if (ro.whole) w += (size_t)(head < H ? head : head - H) * D;
+      else rn = 1.0f / sqrtf(ss / (float)D + eps);
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         u[e] *= rn * (w != nullptr ? to_f(w[4 * l + e]) : 1.0f);
         v[e] *= rn * (w != nullptr ? to_f(w[half + 4 * l + e]) : 1.0f);
+      }
+    }
+    if (head < H && ro.t_every > 0) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { u[e] *= temp; v[e] *= temp; }
+    }
+    if (is_v && ro.v_first != nullptr) {
+      const float lam = *ro.lam;
+      const __nv_bfloat16* fs = reinterpret_cast<const __nv_bfloat16*>(ro.v_first) + (size_t)t * ro.ld_first +
+                                (size_t)(head - H - G) * Dv + 4 * l;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        u[e] = (1.0f - lam) * u[e] + lam * to_f(fs[e]);
+        v[e] = (1.0f - lam) * v[e] + lam * to_f(fs[half + e]);
       }
     }
     const float* ang = is_v ? (v_angles != nullptr ? v_angles + (size_t)t * Dv : nullptr)
@@ -360,15 +435,19 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ o, int n, cons
   }
 }
 
-// `block` > 0: gate and up columns alternate in blocks of that many (the layout of the tcgen05 GEMM's gated epilogue)
+// act 0: silu(gate) * up; 1: gelu(gate) * up, the tanh form. `block` > 0: gate and up columns alternate in blocks of that
+// many (the layout of the tcgen05 GEMM's gated epilogue)
 template <typename T>
 __global__ void silu_mul_kernel(const T* __restrict__ gu, long ld, int F, T* __restrict__ out, long ldo,
-                                size_t total, int block) {
+                                size_t total, int block, int act) {
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= total) return;
   const size_t t = i / F, f = i - t * F;
   const size_t g = block > 0 ? f / block * (2 * block) + f % block : f, u = block > 0 ? g + block : F + f;
-  out[t * ldo + f] = from_f<T>(silu_f(to_f(gu[t * ld + g])) * to_f(gu[t * ld + u]));
+  const float z = to_f(gu[t * ld + g]);
+  const float a = act == 0 ? silu_f(z)
+                           : 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  out[t * ldo + f] = from_f<T>(a * to_f(gu[t * ld + u]));
 }
 
 // Router logits for small batches: one warp per (token, expert), lanes over the width in a fixed order, fp32 result.
@@ -700,8 +779,18 @@ GLLM_EXPORT int gllm_seq_qk_norm_rope_kv_write(const void* qkv, long ld, int nto
                                                int rot, double log2_base, void* q_out, void* kc, void* vc,
                                                const void* slots, int ps, int slab, int slab_v, int is_f32,
                                                const void* freqs, float mag, int unit, const void* angles,
-                                               const void* v_angles, void* stream) {
+                                               const void* v_angles, int whole, float t_coef, int t_every,
+                                               const void* v_first, long ld_first, const void* lam, void* stream) {
   if (ntok <= 0) return 0;
+  if (whole && (unit || qn == nullptr || kn == nullptr || G <= 0)) return 2;
+  if (v_first != nullptr && lam == nullptr) return 2;
+  RowOptions ro;
+  ro.whole = whole;
+  ro.t_coef = t_coef;
+  ro.t_every = t_every;
+  ro.v_first = v_first;
+  ro.ld_first = ld_first;
+  ro.lam = (const float*)lam;
   cudaStream_t st = (cudaStream_t)stream;
   dim3 grid(ntok);
   {
@@ -714,7 +803,7 @@ GLLM_EXPORT int gllm_seq_qk_norm_rope_kv_write(const void* qkv, long ld, int nto
       rope_kv_write_vec_kernel<<<grid, 256, 0, st>>>(
           (const bf16_t*)qkv, ld, H, G, D, Dv, (const bf16_t*)qn, (const bf16_t*)kn, eps, (bf16_t*)q_out, (bf16_t*)kc,
           (bf16_t*)vc, (const int*)slots, ps, slab, slab_v, mag, unit, rot > 0 ? (const float*)angles : nullptr,
-          (const float*)v_angles, (D > Dv ? D : Dv) / 8);
+          (const float*)v_angles, (D > Dv ? D : Dv) / 8, (const int*)positions, ro);
       CUDA_CHECK_RET(cudaGetLastError());
       return 0;
     }
@@ -725,12 +814,12 @@ GLLM_EXPORT int gllm_seq_qk_norm_rope_kv_write(const void* qkv, long ld, int nto
                     (const bf16_t*)qkv, ld, H, G, D, Dv, (const bf16_t*)qn, (const bf16_t*)kn, eps,
                     (const int*)positions, rot, log2_base, (bf16_t*)q_out, (bf16_t*)kc, (bf16_t*)vc,
                     (const int*)slots, ps, slab, slab_v, (const double*)freqs, mag, unit, (const float*)angles,
-                    (const float*)v_angles)),
+                    (const float*)v_angles, ro)),
                 (qk_norm_rope_kv_write_kernel<float><<<grid, 256, smem, st>>>(
                     (const float*)qkv, ld, H, G, D, Dv, (const float*)qn, (const float*)kn, eps,
                     (const int*)positions, rot, log2_base, (float*)q_out, (float*)kc, (float*)vc, (const int*)slots,
                     ps, slab, slab_v, (const double*)freqs, mag, unit, (const float*)angles,
-                    (const float*)v_angles)));
+                    (const float*)v_angles, ro)));
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
 }
@@ -785,15 +874,17 @@ GLLM_EXPORT int gllm_seq_gated_group_norm(const void* o, int n, const void* gate
 }
 
 GLLM_EXPORT int gllm_seq_silu_mul(const void* gu, long ld, int ntok, int F, void* out, long ldo, int is_f32,
-                                  int block, void* stream) {
+                                  int block, int act, void* stream) {
   if (ntok <= 0 || F <= 0) return 0;
   if (block > 0 && F % block != 0) return 2;
   cudaStream_t st = (cudaStream_t)stream;
   const size_t total = (size_t)ntok * F;
   const unsigned blocks = (unsigned)((total + 255) / 256);
   GLLM_BY_DTYPE(is_f32,
-                (silu_mul_kernel<bf16_t><<<blocks, 256, 0, st>>>((const bf16_t*)gu, ld, F, (bf16_t*)out, ldo, total, block)),
-                (silu_mul_kernel<float><<<blocks, 256, 0, st>>>((const float*)gu, ld, F, (float*)out, ldo, total, block)));
+                (silu_mul_kernel<bf16_t><<<blocks, 256, 0, st>>>((const bf16_t*)gu, ld, F, (bf16_t*)out, ldo, total, block,
+                                                                 act)),
+                (silu_mul_kernel<float><<<blocks, 256, 0, st>>>((const float*)gu, ld, F, (float*)out, ldo, total, block,
+                                                               act)));
   CUDA_CHECK_RET(cudaGetLastError());
   return 0;
 }

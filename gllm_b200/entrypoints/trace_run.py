@@ -100,9 +100,9 @@ def _require_kernels(model_dir: str):
     except OSError:
         return
     arch = cfg.get("architecture")
-    if arch in ("Saritar", "Femolix", "Bevovik", "Notadra", "Vikupel"):
+    if arch in ("Saritar", "Femolix", "Bevovik", "Notadra", "Vikupel", "Liverax"):
         from gllm_b200.ops import lib
-        lib.require({"seq", "gemm", "attn"} | (set() if arch == "Vikupel" else {"moe"}))
+        lib.require({"seq", "gemm", "attn"} | (set() if arch in ("Vikupel", "Liverax") else {"moe"}))
 
 
 def main(argv=None) -> int:

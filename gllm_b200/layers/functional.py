@@ -27,10 +27,11 @@ def linear(x, w, bias=None, out=None):
     return ref.linear(x, w, bias)
 
 
-def linear_silu_mul(x, w_interleaved, out=None):
+def linear_silu_mul(x, w_interleaved, out=None, act="silu"):
+    """act(gate) * up of one gate / up projection (rows interleaved per 128); `act`: "silu" | "gelu" (tanh form)."""
     if x.is_cuda:
-        return _sm().linear_silu_mul(x, w_interleaved, out)
-    y = ref.linear_silu_mul(x, w_interleaved)
+        return _sm().linear_silu_mul(x, w_interleaved, out, act=act)
+    y = ref.linear_silu_mul(x, w_interleaved, act=act)
     return y if out is None else out.copy_(y)
 
 
@@ -128,9 +129,9 @@ def embedding_scaled(ids, table, scale):
 
 
 def resid_norm(x, y, w_post, add, w_pre, eps, out_dtype, emit_plain=False, post_scale=None, w_offset=0.0,
-               out_mul=1.0, y_mul=1.0):
+               out_mul=1.0, y_mul=1.0, center=False):
     fn = _seq().resid_norm if x.is_cuda else ref.resid_norm
-    return fn(x, y, w_post, add, w_pre, eps, out_dtype, emit_plain, post_scale, w_offset, out_mul, y_mul)
+    return fn(x, y, w_post, add, w_pre, eps, out_dtype, emit_plain, post_scale, w_offset, out_mul, y_mul, center)
 
 
 def qk_norm_kv_write(qk, num_heads, num_kv_heads, dim, q_norm_w, k_norm_w, eps, k_cache, v_cache, slots):
@@ -183,14 +184,15 @@ def postnorm(x, y, alpha, w, eps, out_dtype):
 
 def qk_norm_rope_kv_write(qkv, num_heads, num_kv_heads, dim, v_dim, q_norm_w, k_norm_w, eps, positions, rot_dims,
                           rot_base, k_cache, v_cache, slots, freqs=None, mag=1.0, unit_norm=False, angles=None,
-                          v_angles=None):
+                          v_angles=None, whole_norm=False, q_temp=None, v_mix=None):
     """num_kv_heads == 0: the rows hold queries only (keys and values are another layer's); `freqs` (fp64 per
     pair) and `mag`: scaled rotary frequencies and the factor on cos / sin. `unit_norm`: q / k divided by their root
     mean square per head, no weight. `angles` (`rotary_angles`): the rows' cos / sin, formed once per step instead of
-    in every layer; `v_angles`: rotate the values over their whole width as well."""
+    in every layer; `v_angles`: rotate the values over their whole width as well. `whole_norm`, `q_temp`, `v_mix`: see
+    `ops.ref.qk_norm_rope_kv_write`."""
     fn = _seq().qk_norm_rope_kv_write if qkv.is_cuda else ref.qk_norm_rope_kv_write
     return fn(qkv, num_heads, num_kv_heads, dim, v_dim, q_norm_w, k_norm_w, eps, positions, rot_dims, rot_base,
-              k_cache, v_cache, slots, freqs, mag, unit_norm, angles, v_angles)
+              k_cache, v_cache, slots, freqs, mag, unit_norm, angles, v_angles, whole_norm, q_temp, v_mix)
 
 
 def rotary_angles(positions, freqs):
@@ -199,20 +201,22 @@ def rotary_angles(positions, freqs):
 
 
 def masked_attention(q, k_cache, v_cache, inp, scale, num_q_heads, head_dim, v_dim, window=None, chunk=None, sink=None,
-                     out_scale=1.0, out=None, softcap=0.0, dist_bias=None, gate=None, v_turn=None):
+                     out_scale=1.0, out=None, softcap=0.0, dist_bias=None, gate=None, v_turn=None, dist_table=None):
     """Paged causal attention with a sliding window and / or a chunk mask, values of their own width, an optional
     per-head sink logit in the denominator and an optional tanh cap on the scaled scores. `dist_bias` (r1, r2):
     r1[h] ln(1 + r2[h] (i - j)) off the scores; `v_turn`: the results of rotated values turned back by the query's
-    angle; `gate`: results times sigmoid(gate)."""
+    angle; `gate`: results times sigmoid(gate); `dist_table` [n, H]: row min(i - j, n - 1) added to the scores."""
     if q.is_cuda:
         return _seq().window_attention(q, k_cache, v_cache, inp.block_table, inp.seq_lens, inp.query_start_loc,
                                        inp.positions, scale, num_q_heads, head_dim, window, sink,
                                        num_decode_seqs=inp.padded_tokens or inp.num_decode_seqs,
                                        max_q_len=inp.max_q_len, chunk=chunk, v_dim=v_dim, out_scale=out_scale, out=out,
-                                       softcap=softcap, dist_bias=dist_bias, gate=gate, v_turn=v_turn)
+                                       softcap=softcap, dist_bias=dist_bias, gate=gate, v_turn=v_turn,
+                                       dist_table=dist_table)
     return ref.window_attention(q, k_cache, v_cache, inp.block_table, inp.seq_lens, inp.query_start_loc, scale,
                                 num_q_heads, head_dim, window, sink, chunk=chunk, v_dim=v_dim, out_scale=out_scale,
-                                out=out, softcap=softcap, dist_bias=dist_bias, gate=gate, v_turn=v_turn)
+                                out=out, softcap=softcap, dist_bias=dist_bias, gate=gate, v_turn=v_turn,
+                                dist_table=dist_table)
 
 
 def linear_state_scan(q, k, v, beta, a, neg_a, dt_bias, decay, state, inp, heads, qk_heads, dim, v_dim, silu_in,
@@ -228,13 +232,15 @@ def gated_group_norm(o, gate, w, group, eps, act, out_scale=1.0, out=None, out_d
     return fn(o, gate, w, group, eps, act, out_scale, out, out_dtype)
 
 
-def silu_mul(gu, out=None, block=0):
-    """silu(gate) * up of [gate | up] rows; `block` > 0: blocks of that many gate and up columns alternate."""
+def silu_mul(gu, out=None, block=0, act="silu"):
+    """act(gate) * up of [gate | up] rows, `act` "silu" | "gelu" (tanh form); `block` > 0: blocks of that many gate and
+    up columns alternate."""
     if gu.is_cuda:
-        if gu.dtype == torch.bfloat16 and gu.is_contiguous() and out is None and not block:
+        if gu.dtype == torch.bfloat16 and gu.is_contiguous() and out is None and not block and act == "silu":
             return _sm().silu_and_mul(gu)
-        return _seq().silu_mul(gu, out, block)
-    return ref.silu_mul(gu, block) if out is None else out.copy_(ref.silu_mul(gu, block))
+        return _seq().silu_mul(gu, out, block, act)
+    y = ref.silu_mul(gu, block, act)
+    return y if out is None else out.copy_(y)
 
 
 def router_topk(h, w, top_k):
@@ -291,16 +297,25 @@ def rglru_scan(u, gates, gate_bias, c_decay, y_pre, y_bias, state, inp, block, o
                           inp.query_start_loc, block, out_dtype)
 
 
-def latent_norm_rope_write(q, dkv, rank, rot, norm_w, eps, positions, freqs, mag, q_full, cache, slots):
+def latent_norm_rope_write(q, dkv, rank, rot, norm_w, eps, positions, freqs, mag, q_full, cache, slots, angles=None):
+    """`angles` (`rotary_angles`): pairs (i, i + rot / 2) turned by the step's cos / sin rows; without it neighbouring
+    pairs, the angle formed from `freqs` in the kernel."""
     fn = _lat().latent_norm_rope_write if q.is_cuda else ref.latent_norm_rope_write
-    return fn(q, dkv, rank, rot, norm_w, eps, positions, freqs, mag, q_full, cache, slots)
+    return fn(q, dkv, rank, rot, norm_w, eps, positions, freqs, mag, q_full, cache, slots, angles)
 
 
-def latent_attention(q_full, cache, inp, scale, rank):
-    """Causal multi-query attention over the paged latent cache (values = the first `rank` columns of the keys)."""
+def latent_attention(q_full, cache, inp, scale, rank, window=None, sink=None):
+    """Causal multi-query attention over the paged latent cache (values = the first `rank` columns of the keys), with
+    an optional sliding window and per-head softmax sink."""
     if q_full.is_cuda:
-        return _lat().latent_attention(q_full, cache, inp, scale, rank)
-    return ref.latent_attention(q_full, cache, inp.block_table, inp.seq_lens, inp.query_start_loc, scale, rank)
+        return _lat().latent_attention(q_full, cache, inp, scale, rank, window=window, sink=sink)
+    return ref.latent_attention(q_full, cache, inp.block_table, inp.seq_lens, inp.query_start_loc, scale, rank, window,
+                                sink)
+
+
+def gate_rows(o, gate):
+    """In place: o [T, n] times sigmoid(gate [T, n]) (any row stride)."""
+    return _lat().gate_rows(o, gate) if o.is_cuda else ref.gate_rows(o, gate)
 
 
 def grouped_router(h, w, correction, top_k, n_groups, keep_groups, scale, score="softmax", group_top=1, renorm=True):

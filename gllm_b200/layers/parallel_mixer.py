@@ -45,9 +45,9 @@ class CoreMixer(nn.Module):
         n_in_pad = self.n_in_pad + 2 * self.ff
         self.in_w = nn.Parameter(torch.zeros(n_in_pad, hidden, dtype=dtype, device=device), requires_grad=False)
         self.o_w = nn.Parameter(torch.zeros(hidden, self.n_joint, dtype=dtype, device=device), requires_grad=False)
-        # biases of the input projection ('<projection>.b'), for cores that declare `has_bias`; rows of others stay 0
+        # biases of the input projection ('<projection>.b'), for cores that declare them (`bias_names`); other rows stay 0
         self.in_b = nn.Parameter(torch.zeros(n_in_pad, dtype=dtype, device=device), requires_grad=False) \
-            if any(getattr(c, "has_bias", False) for c in cores) else None
+            if any(getattr(c, "bias_names", ()) for c in cores) else None
         self.uses_pages = any(c.uses_pages for c in cores)
         self.uses_state = any(c.uses_state for c in cores)
 
@@ -86,7 +86,7 @@ class CoreMixer(nn.Module):
                 t = reader.get(p + n)
                 assert t.shape[0] == r, (p + n, tuple(t.shape), r)
                 rows.append(t)
-                if getattr(c, "has_bias", False):
+                if n in getattr(c, "bias_names", ()):
                     b = reader.get(p + n + ".b")
                     assert tuple(b.shape) == (r,), (p + n + ".b", tuple(b.shape), r)
                     self.in_b.data[at:at + r].copy_(b)

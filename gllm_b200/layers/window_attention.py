@@ -75,9 +75,18 @@ class RotaryChunkCore(nn.Module):
         frequencies of `rot_base` over v_dim, unscaled) and cached so; the result at position i is turned back by i;
       * `dist_bias`: r1[h] ln(1 + r2[h] (i - j)) is taken off the scaled score (per-head numbers 'r1', 'r2');
       * `out_gate`: the heads' results are multiplied by sigmoid of one more projection of the input ('g');
-      * `rot_scaling` with {factor, low, high, original}: the frequency bands of `ops.ref.banded_rotary_frequencies`.
-    With `unit_qk` or `turn_values` the cos / sin rows come from `inp.angles` (formed once per step by the model, see
-    `angle_tables`) instead of from every layer's own kernel.
+      * `rot_scaling` with {factor, low, high, original}: the frequency bands of `ops.ref.banded_rotary_frequencies`;
+        with a factor alone every frequency is divided by it;
+      * `whole_norm`: the RMS norms of q and k run over the whole projection, before it is split into heads (weights
+        'q.norm' [heads * dim], 'k.norm' [kv_heads * dim]);
+      * `q_temp` (coef, every): the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1), after
+        norm and rotation;
+      * `dist_rows`, `dist_max`: a learned bias per head and distance bucket ('rel' [rows, heads], buckets of
+        `ops.ref.distance_buckets`) is added to the scaled scores; kept expanded to one fp32 row per distance;
+      * `v_mix`: every core with it but the first one to run in a step caches (1 - lam) v + lam v_first, v_first the
+        first one's values of the same tokens (`inp.first_values`), lam a learned number ('vmix').
+    With `unit_qk`, `turn_values`, bands or a linear scaling (or on request, `step_angles`) the cos / sin rows come from
+    `inp.angles` (formed once per step by the model, see `angle_tables`) instead of from every layer's own kernel.
     A core in the sense of layers/parallel_mixer.py: it reads [q | k | v] rows of a joint projection."""
     uses_pages, uses_state = True, False
 
@@ -85,14 +94,15 @@ class RotaryChunkCore(nn.Module):
                  chunk: Optional[int], window: Optional[int], eps: float, dtype, device, qk_norm: bool = True,
                  rot_scaling: Optional[dict] = None, softcap: float = 0.0, unit_sink: bool = False,
                  bias: bool = False, kv_from: Optional[int] = None, unit_qk: bool = False, turn_values: bool = False,
-                 dist_bias: bool = False, out_gate: bool = False):
+                 dist_bias: bool = False, out_gate: bool = False, whole_norm: bool = False, q_temp=None,
+                 dist_rows: int = 0, dist_max: float = 0.0, v_mix: bool = False, step_angles: bool = False):
         super().__init__()
         assert heads % kv_heads == 0, (heads, kv_heads)
         assert rot_dims % 2 == 0 and rot_dims <= dim, (rot_dims, dim)
         self.heads, self.kv_heads, self.dim, self.v_dim = heads, kv_heads, dim, v_dim
         self.scale, self.rot_dims, self.rot_base, self.chunk, self.window, self.eps = \
             float(scale), int(rot_dims), float(rot_base), chunk, window, eps
-        self.softcap, self.has_bias, self.kv_from = float(softcap or 0.0), bool(bias), kv_from
+        self.softcap, self.kv_from = float(softcap or 0.0), kv_from
         if kv_from is None:
             self.in_names = ("q", "k", "v")
             self.in_rows = (heads * dim, kv_heads * dim, kv_heads * v_dim)
@@ -100,6 +110,11 @@ class RotaryChunkCore(nn.Module):
             self.in_names = ("q",)
             self.in_rows = (heads * dim,)
         self.unit_qk, self.turn_values, self.out_gate = bool(unit_qk), bool(turn_values), bool(out_gate)
+        self.bias_names = self.in_names if bias else ()
+        self.whole_norm = bool(whole_norm)
+        self.q_temp = (float(q_temp[0]), int(q_temp[1])) if q_temp is not None else None
+        assert not whole_norm or (qk_norm and kv_from is None)
+        assert kv_from is None or (q_temp is None and not v_mix)
         assert not (unit_qk and qk_norm) and not ((unit_qk or turn_values) and kv_from is not None)
         assert not turn_values or v_dim % 2 == 0, v_dim
         if out_gate:
@@ -111,13 +126,24 @@ class RotaryChunkCore(nn.Module):
         else:
             self.r1 = self.r2 = None
         self.n_in, self.n_out = sum(self.in_rows), heads * v_dim
-        self.q_norm_w = nn.Parameter(torch.zeros(dim, dtype=dtype, device=device), requires_grad=False) if qk_norm \
-            else None
-        self.k_norm_w = nn.Parameter(torch.zeros(dim, dtype=dtype, device=device), requires_grad=False) if qk_norm \
-            else None
+
+        def par(n, dt=dtype):
+            return nn.Parameter(torch.zeros(n, dtype=dt, device=device), requires_grad=False)
+
+        self.q_norm_w = par(heads * dim if whole_norm else dim) if qk_norm else None
+        self.k_norm_w = par(kv_heads * dim if whole_norm else dim) if qk_norm else None
+        self.vmix = par(1, torch.float32) if v_mix else None
         self.mag = 1.0
         from gllm_b200.ops import ref
-        self.step_angles = self.unit_qk or self.turn_values or bool(rot_scaling and "low" in rot_scaling)
+        if dist_rows:
+            assert not dist_bias
+            self.dist_rows, self.buckets = int(dist_rows), ref.distance_buckets(int(dist_rows), float(dist_max))
+            self.dist_table = nn.Parameter(torch.zeros(len(self.buckets), heads, dtype=torch.float32, device=device),
+                                           requires_grad=False)
+        else:
+            self.dist_table = None
+        self.step_angles = bool(step_angles) or self.unit_qk or self.turn_values or \
+            bool(rot_scaling and ("low" in rot_scaling or "original" not in rot_scaling))
         if self.step_angles:
             self.register_buffer("freqs", ref.banded_rotary_frequencies(rot_dims, rot_base, rot_scaling).to(device),
                                  persistent=False)
@@ -167,17 +193,27 @@ class RotaryChunkCore(nn.Module):
             return out
         kc, vc = cache.k_cache[run_id], cache.v_cache[run_id]
         own = self.kv_from is None
-        if self.step_angles or self.r1 is not None or self.out_gate:
+        v_mix = None
+        if self.vmix is not None:
+            v = proj[:, (self.heads + self.kv_heads) * self.dim:][:, :self.kv_heads * self.v_dim]
+            if getattr(inp, "first_values", None) is None:
+                inp.first_values = v
+            else:
+                v_mix = (inp.first_values, self.vmix)
+        if self.step_angles or self.r1 is not None or self.out_gate or self.whole_norm or self.q_temp is not None or \
+                self.vmix is not None or self.dist_table is not None:
             ang = self._angles(inp, "freqs") if self.step_angles else None
             v_ang = self._angles(inp, "v_freqs") if self.step_angles else None
             q = Fn.qk_norm_rope_kv_write(proj, self.heads, self.kv_heads if own else 0, self.dim, self.v_dim,
                                          self.q_norm_w, self.k_norm_w, self.eps, inp.positions, self.rot_dims,
                                          self.rot_base, kc, vc, inp.slot_mapping, None if self.step_angles
-                                         else self.freqs, self.mag, self.unit_qk, ang, v_ang)
+                                         else self.freqs, self.mag, self.unit_qk, ang, v_ang, self.whole_norm,
+                                         self.q_temp, v_mix)
             gate = proj[:, self.n_in - self.n_out:self.n_in] if self.out_gate else None
             return Fn.masked_attention(q, kc, vc, inp, self.scale, self.heads, self.dim, self.v_dim, self.window,
                                        self.chunk, self.sink, out_scale, out, self.softcap,
-                                       (self.r1, self.r2) if self.r1 is not None else None, gate, v_ang)
+                                       (self.r1, self.r2) if self.r1 is not None else None, gate, v_ang,
+                                       self.dist_table)
         q = Fn.qk_norm_rope_kv_write(proj, self.heads, self.kv_heads if own else 0, self.dim, self.v_dim,
                                      self.q_norm_w, self.k_norm_w, self.eps, inp.positions, self.rot_dims,
                                      self.rot_base, kc, vc, inp.slot_mapping, self.freqs, self.mag)
@@ -191,3 +227,9 @@ class RotaryChunkCore(nn.Module):
         if getattr(self, "r1", None) is not None:
             put(self.r1, reader.get(pre + "r1").float())
             put(self.r2, reader.get(pre + "r2").float())
+        if self.vmix is not None:
+            put(self.vmix, reader.get(pre + "vmix").float().reshape(1))
+        if self.dist_table is not None:
+            rel = reader.get(pre + "rel")
+            assert rel.shape[0] == self.dist_rows, (tuple(rel.shape), self.dist_rows)
+            put(self.dist_table, rel.float()[torch.tensor(self.buckets)])

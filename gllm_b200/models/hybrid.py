@@ -12,7 +12,16 @@ sigmoid-scored, group-limited mixture of ungated squared-ReLU experts; a hashed 
 token pair added to the token embedding; logits scaled through the final norm); and parallel blocks (architecture
 `Vikupel`: Mamba-2 mixers, windowed attention with a logarithmic distance bias and an output gate, rotary attention with
 rotated values, gated SiLU feed-forward beside the mixer, a residual multiplier, a gated per-layer token embedding after
-every layer, a loop whose passes share weights).
+every layer, a loop whose passes share weights); and pre-norm blocks with layer norms (architecture `Liverax`: rotary
+window attention, attention with a bucketed distance bias, norms over whole projections, a query temperature and an output
+gate, windowed latent attention with a sink and an output gate, values mixed with the first mixing layer's, gated tanh-gelu
+feed-forward, capped logits).
+
+The pre-norm form (the sandwich form without the norms behind the sublayers; ln: layer norm without a bias):
+
+    x = embed[token]
+    per layer:  x += mixer(ln(x) * n1) ;  x += ff(ln(x) * n2)                            (second line only with a ff)
+    logits = cap * tanh(head @ (ln(x) * final_norm) / cap)
 
 The branch-norm form:
 
@@ -63,11 +72,12 @@ x += mult * y in one kernel that also emits x in the compute dtype for G; the se
 multiplier, next layer's norm1) is one kernel as in the sandwich form.
 
 config.json keys read here: architecture, vocab, width, residual_mult, token_side.dim, embedding.scale, embedding.bigram.{buckets, mul_prev,
-mul_cur}, logit_scale, layers[i].mixer.{kv_from, softcap, rot.scaling.{factor, original, fast, slow}},
+mul_cur}, logit_scale, layers[i].mixer.{kv_from, softcap, rot.scaling.{factor, original, fast, slow}, bias_max, q_temp.{coef,
+every}, v_mix, mask.size},
 norm.eps, loop.{start,stop,times},
 postln_alpha, logit_softcap, layers[i].{type, mixer{...}, mlp{kind, ff | expert.{ff, limit}, router.{experts, top,
 identity, scale, groups.{count, keep}}, shared.{ff, limit}} | null}, optional torch_dtype. Tensor names: embed, bigram,
-head, side.embed, l<i>.side.{gate,proj,norm}, l<i>.mix.{q,k,v}.b, l<i>.mlp.e<j>.{up,down}, final.norm, l<i>.norm1|norm1b|norm2|norm2b|ls1|ls2, l<i>.mix.*, l<i>.mlp.up|down|gate|router|correction|
+head, side.embed, l<i>.side.{gate,proj,norm}, l<i>.mix.{q,k,v}.b, l<i>.mix.{rel,vmix,g,sink}, l<i>.mlp.e<j>.{up,down}, final.norm, l<i>.norm1|norm1b|norm2|norm2b|ls1|ls2, l<i>.mix.*, l<i>.mlp.up|down|gate|router|correction|
 e<j>.{gate,up,down}|shared.{gate,up,down}.
 """
 from __future__ import annotations
@@ -104,13 +114,14 @@ class HybridSpec:
     loop_times: int = 1
     dtype: torch.dtype = torch.bfloat16
     # "sandwich": x += post(f(pre(x))) | "postnorm": x <- norm(alpha x + f(x)) | "branchnorm": x += ls * post(f(x)) |
-    # "parallel": x += mult (mixer(pre(x)) + ff(pre(x)))
+    # "parallel": x += mult (mixer(pre(x)) + ff(pre(x))) | "prenorm": x += f(pre(x))
     block: str = "sandwich"
     resid_alpha: float = 1.0
     logit_softcap: float = 0.0         # 0: none
     # "relu2": down(relu(up h)^2) | "silu_gate": down(silu(gate h) * up h) | "glu_clamp": clamped gate and up,
-    # down(g sigmoid(1.702 g) (u + 1))
+    # down(g sigmoid(1.702 g) (u + 1)) | "gelu_gate": down(gelu_tanh(gate h) * up h)
     ff_act: str = "relu2"
+    center_norm: bool = False          # the pre-norms are layer norms without a bias instead of RMS norms
     norm_offset: float = 0.0           # added to every norm weight in fp32 (1.0: weights stored around zero)
     logit_scale: float = 1.0
     # {"buckets", "mul_prev", "mul_cur"}: a second embedding table indexed by a hash of the (previous, current) pair
@@ -186,6 +197,16 @@ def spec_vikupel(cfg) -> HybridSpec:
                       token_side_dim=int(side.get("dim", 0)), eos_token_id=cfg.get("eos_token_id"))
 
 
+def spec_liverax(cfg) -> HybridSpec:
+    dt = cfg.get("torch_dtype", cfg.get("dtype", "bfloat16"))
+    if dt not in _DTYPES:
+        raise ValueError(f"unsupported dtype {dt} for this architecture (bfloat16 | float32)")
+    return HybridSpec(arch="liverax", hidden_size=int(cfg["width"]), vocab_size=int(cfg["vocab"]),
+                      rms_eps=float(cfg["norm"]["eps"]), embed_scale=1.0, layers=[dict(x) for x in cfg["layers"]],
+                      dtype=_DTYPES[dt], block="prenorm", center_norm=True, ff_act="gelu_gate",
+                      logit_softcap=float(cfg.get("logit_softcap") or 0.0), eos_token_id=cfg.get("eos_token_id"))
+
+
 def layer_runs(n_layers: int, start: int, stop: int, times: int, readd: bool = True):
     """[(layer index, add_embed)] in execution order; add_embed marks the first layer of every pass but the first
     (never without `readd`)."""
@@ -229,8 +250,37 @@ def make_parallel_mixer(kind: str, m: dict, ff: int, spec: HybridSpec, device):
     return CoreMixer(h, [core], [""], [1.0], dt, device, ff=ff)
 
 
+def make_prenorm_mixer(kind: str, m: dict, spec: HybridSpec, device):
+    h, dt, eps = spec.hidden_size, spec.dtype, spec.rms_eps
+    rot, window = m.get("rot") or {}, (m.get("mask") or {}).get("size")
+    window = int(window) if window is not None else None
+    if kind == "attention":            # rotary, sliding window
+        core = RotaryChunkCore(int(m["heads"]), int(m.get("kv_heads", m["heads"])), int(m["dim"]),
+                               int(m.get("vdim", m["dim"])), float(m["scale"]), int(rot.get("dims", m["dim"])),
+                               float(rot.get("base", 10000.0)), None, window, eps, dt, device, qk_norm=False,
+                               rot_scaling=rot.get("scaling"), v_mix=bool(m.get("v_mix")), step_angles=True)
+    elif kind == "attention_2":        # no rotation, norms over whole projections, bucketed distance bias, output gate
+        qt = m.get("q_temp")
+        core = RotaryChunkCore(int(m["heads"]), int(m.get("kv_heads", m["heads"])), int(m["dim"]),
+                               int(m.get("vdim", m["dim"])), float(m["scale"]), 0, 10000.0, None, window, eps, dt, device,
+                               whole_norm=True, bias=True, out_gate=True, v_mix=bool(m.get("v_mix")),
+                               q_temp=(qt["coef"], qt["every"]) if qt else None, dist_rows=int(m["bias_rows"]),
+                               dist_max=float(m["bias_max"]))
+    elif kind == "latent_attention":
+        rd = int(m.get("rot_dim", rot.get("dims", 0)))
+        assert int(rot.get("dims", rd)) == rd, "the rotated part is rotated whole"
+        return LatentAttention(h, int(m["heads"]), int(m["dim"]), rd, int(m.get("vdim", m["dim"])), int(m["q_rank"]),
+                               int(m["kv_rank"]), float(m["scale"]), float(rot.get("base", 10000.0)), rot.get("scaling"),
+                               eps, dt, device, half_split=True, window=window, use_sink=True, out_gate=True)
+    else:
+        raise ValueError(f"unknown mixer type {kind!r}")
+    return CoreMixer(h, [core], [""], [1.0], dt, device)
+
+
 def make_mixer(kind: str, m: dict, spec: HybridSpec, device):
     h, dt = spec.hidden_size, spec.dtype
+    if spec.block == "prenorm":
+        return make_prenorm_mixer(kind, m, spec, device)
     if spec.block == "parallel":
         return make_parallel_mixer(kind, m, 0, spec, device)
     if kind == "attention" and spec.arch == "notadra":
@@ -282,12 +332,13 @@ def make_mixer(kind: str, m: dict, spec: HybridSpec, device):
 
 
 class GatedMLP(nn.Module):
-    """down(silu(gate h) * (up h)); gate and up rows share one GEMM. On CUDA in bf16 with ff % 128 == 0 the rows are
-    stored interleaved per 128 and the product is the tcgen05 GEMM's SiLU-gate epilogue (one kernel)."""
+    """down(act(gate h) * (up h)), act silu or gelu (tanh form); gate and up rows share one GEMM. On CUDA in bf16 with
+    ff % 128 == 0 the rows are stored interleaved per 128 and the product is the tcgen05 GEMM's gated epilogue (one
+    kernel)."""
 
-    def __init__(self, hidden: int, ff: int, dtype, device):
+    def __init__(self, hidden: int, ff: int, dtype, device, act: str = "silu"):
         super().__init__()
-        self.ff = ff
+        self.ff, self.act = ff, act
         self.fused = torch.device(device).type == "cuda" and dtype == torch.bfloat16 and ff % 128 == 0 and \
             hidden % 8 == 0
         self.gate_up_w = nn.Parameter(torch.zeros(2 * ff, hidden, dtype=dtype, device=device), requires_grad=False)
@@ -301,14 +352,16 @@ class GatedMLP(nn.Module):
 
     def forward(self, h):
         if self.fused:
-            return Fn.linear_any(Fn.linear_silu_mul(h, self.gate_up_w), self.down_w)
-        return Fn.linear_any(Fn.silu_mul(Fn.linear_any(h, self.gate_up_w)), self.down_w)
+            return Fn.linear_any(Fn.linear_silu_mul(h, self.gate_up_w, act=self.act), self.down_w)
+        return Fn.linear_any(Fn.silu_mul(Fn.linear_any(h, self.gate_up_w), act=self.act), self.down_w)
 
 
 def make_ff(mlp: dict, spec: HybridSpec, device):
     h, dt = spec.hidden_size, spec.dtype
     kind = mlp.get("kind", "dense")
     if kind == "dense":
+        if spec.ff_act == "gelu_gate":
+            return GatedMLP(h, int(mlp["ff"]), dt, device, act="gelu")
         return (GatedMLP if spec.ff_act == "silu_gate" else Relu2MLP)(h, int(mlp["ff"]), dt, device)
     if kind == "moe" and spec.ff_act == "relu2":
         r = mlp["router"]
@@ -394,8 +447,11 @@ class HybridLM(nn.Module):
         # cos / sin rows that layers read instead of forming them: one table per distinct set of frequencies and step
         self.angle_tables = {}
         for l in self.layers:
-            for c in getattr(l.mixer, "cores", []):
+            for c in getattr(l.mixer, "cores", [l.mixer]):
                 self.angle_tables.update(dict(c.angle_tables()) if hasattr(c, "angle_tables") else {})
+        mixing = {(c.kv_heads * c.v_dim) for l in self.layers for c in getattr(l.mixer, "cores", [])
+                  if getattr(c, "vmix", None) is not None}
+        assert len(mixing) <= 1, "layers that mix their values with the first one's have values of one width"
         # the pair embedding keeps every sequence's last token in its state slot
         self.has_state = any(getattr(l.mixer, "uses_state", not l.mixer.uses_pages) for l in self.layers) or \
             spec.pair_hash is not None
@@ -440,7 +496,9 @@ class HybridLM(nn.Module):
             return self._forward_branchnorm(inp, cache), None
         if spec.block == "parallel":
             return self._forward_parallel(inp, cache), None
-        off = spec.norm_offset
+        off, center = spec.norm_offset, spec.center_norm
+        inp.angles = {k: Fn.rotary_angles(inp.positions, f) for k, f in self.angle_tables.items()}
+        inp.first_values = None
         if spec.pair_hash is not None:
             ph = spec.pair_hash
             x0 = Fn.embedding_pair_hash(inp, self.embed_w, self.pair_w, ph["mul_prev"], ph["mul_cur"], ph["buckets"],
@@ -451,13 +509,13 @@ class HybridLM(nn.Module):
         n = len(self.runs)
         # the logit scale rides on the final norm (applied in fp32 before the head's input is rounded)
         h = Fn.resid_norm(x, None, None, None, self.layers[self.runs[0][0]].norm1_w if n else self.final_norm_w,
-                          eps, dt, False, None, off, 1.0 if n else spec.logit_scale)
+                          eps, dt, False, None, off, 1.0 if n else spec.logit_scale, center=center)
         for r, (li, _) in enumerate(self.runs):
             L = self.layers[li]
             y = L.mixer(inp, h, cache, r)
             post = L.norm1b_w
             if L.mlp is not None:
-                h = Fn.resid_norm(x, y, post, None, L.norm2_w, eps, dt, False, None, off)
+                h = Fn.resid_norm(x, y, post, None, L.norm2_w, eps, dt, False, None, off, center=center)
                 y = L.mlp(h)
                 post = L.norm2b_w
             last = r + 1 == n
@@ -467,9 +525,10 @@ class HybridLM(nn.Module):
             if self.trace is not None:
                 Fn.resid_norm(x, y, post, None, None, eps, dt, False, None, off)
                 self.trace.append(x.clone())
-                h = Fn.resid_norm(x, None, None, add, w_pre, eps, dt, False, None, off, mul)
+                h = Fn.resid_norm(x, None, None, add, w_pre, eps, dt, False, None, off, mul, center=center)
             else:
-                h = Fn.resid_norm(x, y, post, add, w_pre, eps, dt, False, None, off, mul)
+                h = Fn.resid_norm(x, y, post, add, w_pre, eps, dt, False, None, off, mul, center=center)
+        inp.angles = inp.first_values = None
         return h, None
 
     def _forward_postnorm(self, inp, cache):
@@ -579,6 +638,10 @@ class HybridLM(nn.Module):
                 p.data.copy_(-torch.exp(torch.rand(p.shape, generator=g) * 2.0 - 1.0))
             elif name.endswith("dt_bias"):
                 p.data.copy_(torch.rand(p.shape, generator=g) * 2.0 - 3.0)
+            elif name.endswith("dist_table"):
+                rnd(p, 0.5)
+            elif name.endswith("vmix"):
+                p.data.fill_(0.3)
             elif name.endswith("conv_b") and "cores" in name:
                 p.data.zero_()
             elif name.endswith("sink") or name.endswith("conv_b"):
@@ -695,3 +758,7 @@ def build_notadra(cfg, device):
 
 def build_vikupel(cfg, device):
     return HybridLM(spec_vikupel(cfg), device)
+
+
+def build_liverax(cfg, device):
+    return HybridLM(spec_liverax(cfg), device)

@@ -4,7 +4,7 @@ Supported `architectures[0]` values:
   LlamaForCausalLM, Qwen2ForCausalLM, Qwen3ForCausalLM, Qwen2MoeForCausalLM, Qwen3MoeForCausalLM,
   MixtralForCausalLM, ChatGLMModel / ChatGLMForConditionalGeneration, DeepseekV2ForCausalLM,
   DeepseekV3ForCausalLM, Qwen2_5_VLForConditionalGeneration, Qwen3VLForConditionalGeneration,
-  Qwen3VLMoeForConditionalGeneration, Saritar, Femolix, Bevovik, Notadra and Vikupel (layer-list decoders,
+  Qwen3VLMoeForConditionalGeneration, Saritar, Femolix, Bevovik, Notadra, Vikupel and Liverax (layer-list decoders,
   models/hybrid.py).
 """
 from __future__ import annotations
@@ -182,6 +182,11 @@ def _build_vikupel(cfg, device):
     return build_vikupel(cfg, device)
 
 
+def _build_liverax(cfg, device):
+    from gllm_b200.models.hybrid import build_liverax
+    return build_liverax(cfg, device)
+
+
 def _build_femolix(cfg, device):
     from gllm_b200.models.hybrid import build_femolix
     return build_femolix(cfg, device)
@@ -193,6 +198,7 @@ ARCHITECTURES: Dict[str, Callable] = {
     "Bevovik": _build_bevovik,
     "Notadra": _build_notadra,
     "Vikupel": _build_vikupel,
+    "Liverax": _build_liverax,
     "LlamaForCausalLM": _build_decoder(spec_llama),
     "MistralForCausalLM": _build_decoder(spec_llama),
     "Qwen2ForCausalLM": _build_decoder(spec_qwen2),
@@ -213,7 +219,13 @@ ARCHITECTURES: Dict[str, Callable] = {
 def complete_config(cfg: HFConfig, reader) -> None:
     """Sizes that a config leaves to the checkpoint's tensor shapes are written into `cfg` before the model is
     built (`reader` is None for random weights: defaults apply). Bevovik: the rank of a `gla` mixer's decay
-    projection is the row count of `l<i>.mix.a1`."""
+    projection is the row count of `l<i>.mix.a1`. Liverax: the number of distance buckets of an `attention_2` mixer is the
+    row count of `l<i>.mix.rel`."""
+    if cfg["architectures"][0] == "Liverax":
+        for i, layer in enumerate(cfg.get("layers") or []):
+            m = layer.get("mixer") or {}
+            if layer.get("type") == "attention_2" and "bias_rows" not in m:
+                m["bias_rows"] = int(reader.shape(f"l{i}.mix.rel")[0]) if reader is not None else 32
     if cfg["architectures"][0] == "Bevovik":
         for i, layer in enumerate(cfg.get("layers") or []):
             m = layer.get("mixer") or {}

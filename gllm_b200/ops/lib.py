@@ -64,7 +64,7 @@ def _declare(lib):
     sig("gllm_attn_decode", [P, L, P, P, P, L, P, P, P, P, I, I, I, I, I, I, I, I, F, P, P])
     sig("gllm_attn_prefill", [P, L, P, P, P, L, P, P, P, I, I, I, I, I, I, I, I, F, P])
     sig("gllm_attn_prefill_tc", [P, L, P, P, P, L, P, P, P, I, I, I, I, I, I, I, I, F, I, P])
-    sig("gllm_mla_attention", [P, P, P, L, P, P, P, P, P, I, I, I, I, I, F, P])
+    sig("gllm_mla_attention", [P, P, P, L, P, P, P, P, P, I, I, I, I, I, F, I, P, P])
     sig("gllm_mla_rope_cache", [P, L, L, I, P, P, L, P, L, P, P, P, P, I, I, P])
     sig("gllm_sample", [P, I, L, P, I, I, P, P, P, P, P, I, P, c_uint64, P, P, I, P])
     sig("gllm_mark_seen", [P, I, P, P, I, P])
@@ -76,6 +76,7 @@ def _declare(lib):
     sig("gllm_moe_grouped_gemm", [P, L, P, P, L, I, I, I, I, P, P, I, P, P])
     sig("gllm_moe_grouped_gemm_glu", [P, L, P, P, L, I, I, I, I, P, P, F, F, P])
     sig("gllm_gemm_bf16_glu", [P, L, P, L, P, L, I, I, I, F, F, P, L, P, I, P])
+    sig("gllm_gemm_bf16_gelu", [P, L, P, L, P, L, I, I, I, P, L, P, I, P])
     sig("gllm_moe_combine", [P, P, P, P, I, I, I, P])
     sig("gllm_fp8_quant_group", [P, L, P, P, I, I, P])
     sig("gllm_moe_grouped_gemm_fp8", [P, P, P, P, P, L, I, I, I, I, P, P, I, P])

@@ -8,7 +8,7 @@ hand-written kernels in `gllm_b200.ops.sm100`.
 from __future__ import annotations
 
 import math
-from typing import Optional
+from typing import List, Optional, Tuple
 
 import torch
 import torch.nn.functional as F
@@ -60,11 +60,11 @@ def interleave_gate_up(w: torch.Tensor, block: int = 128) -> torch.Tensor:
     return torch.cat([g, u], dim=1).reshape(two_i, k).contiguous()
 
 
-def linear_silu_mul(x: torch.Tensor, w_interleaved: torch.Tensor, block: int = 128) -> torch.Tensor:
+def linear_silu_mul(x: torch.Tensor, w_interleaved: torch.Tensor, block: int = 128, act: str = "silu") -> torch.Tensor:
     y = F.linear(x, w_interleaved)
     t, two_i = y.shape
     y = y.reshape(t, two_i // (2 * block), 2, block)
-    return (F.silu(y[:, :, 0].float()) * y[:, :, 1].float()).to(x.dtype).reshape(t, two_i // 2)
+    return (_gate_act(y[:, :, 0].float(), act) * y[:, :, 1].float()).to(x.dtype).reshape(t, two_i // 2)
 
 
 def embedding(ids: torch.Tensor, table: torch.Tensor, vocab_start: int = 0, vocab_end: Optional[int] = None):
@@ -467,14 +467,15 @@ def embedding_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float) -> to
 def resid_norm(x: torch.Tensor, y: Optional[torch.Tensor], w_post: Optional[torch.Tensor],
                add: Optional[torch.Tensor], w_pre: Optional[torch.Tensor], eps: float, out_dtype,
                emit_plain: bool = False, post_scale: Optional[torch.Tensor] = None, w_offset: float = 0.0,
-               out_mul: float = 1.0, y_mul: float = 1.0):
+               out_mul: float = 1.0, y_mul: float = 1.0, center: bool = False):
     """In place on the fp32 stream x [T, W]:  x += rms(y) * w_post ;  x += add ;  returns rms(x) * w_pre cast to
     `out_dtype` (None when w_pre is None). Every step is optional. All arithmetic in fp32. `post_scale` [W] fp32
     (a layer scale) multiplies the normed branch element by element: x += rms(y) * w_post * post_scale. `emit_plain` (with w_pre None): returns the stream itself rounded to
     `out_dtype` — x for fp32 — for sublayers that read the stream without a norm in front. `w_offset` is added to
     both norm weights in fp32 (1.0 for weights stored around zero); `out_mul` multiplies the normed result before it
     is rounded (a logit scale folded into the final norm). `y_mul` multiplies the branch before it is added (a residual
-    multiplier); without w_post the branch is added as it is, not normed: x += y_mul * y."""
+    multiplier); without w_post the branch is added as it is, not normed: x += y_mul * y. `center`: the pre-norm is a
+    layer norm without a bias, (x - mean) / sqrt(mean of the squared deviations + eps) * w_pre."""
     if y is not None:
         br = y.float()
         if w_post is not None:
@@ -488,6 +489,8 @@ def resid_norm(x: torch.Tensor, y: Optional[torch.Tensor], w_post: Optional[torc
         if emit_plain:
             return x if out_dtype == torch.float32 else x.to(out_dtype)
         return None
+    if center:
+        x = x - x.mean(-1, keepdim=True)
     return (x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps) * (w_pre.float() + w_offset) * out_mul).to(out_dtype)
 
 
@@ -523,7 +526,8 @@ def window_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      head_dim: int, window: Optional[int], sink: Optional[torch.Tensor],
                      chunk: Optional[int] = None, v_dim: Optional[int] = None, out_scale: float = 1.0,
                      out: Optional[torch.Tensor] = None, softcap: float = 0.0, dist_bias=None,
-                     gate: Optional[torch.Tensor] = None, v_turn: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     gate: Optional[torch.Tensor] = None, v_turn: Optional[torch.Tensor] = None,
+                     dist_table: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal paged attention where position i sees j with 0 <= i - j < window (None: all of the past), and, with
     `chunk`, only j of its own chunk (floor(i / chunk) == floor(j / chunk), counted from position 0); the softmax
     denominator has one more term exp(sink[h]) that carries no value (None: plain softmax). Values may be wider or
@@ -532,7 +536,8 @@ def window_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     mask and the softmax. `dist_bias` = (r1, r2) [H] fp32: r1[h] ln(1 + r2[h] (i - j)) is taken off the score of key j
     for the query at i. `v_turn` [T, v_dim] fp32 (cos | sin per pair, of the query's position): the values were
     rotated by their own positions, and every head's result is turned back, pair (m, m + v_dim / 2) by the negative
-    angle. `gate` [T, H * v_dim] (any row stride): the result is multiplied by sigmoid(gate), last."""
+    angle. `gate` [T, H * v_dim] (any row stride): the result is multiplied by sigmoid(gate), last. `dist_table` [n, H]
+    fp32: row min(i - j, n - 1) is added to the scaled score of key j for the query at i."""
     t = q.shape[0]
     hq, d = num_q_heads, head_dim
     dv = d if v_dim is None else v_dim
@@ -556,6 +561,8 @@ def window_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         if dist_bias is not None:
             r1, r2 = (r.float().view(hq, 1, 1) for r in dist_bias)
             att = att - r1 * torch.log1p(r2 * (qi - kj).clamp(min=0).unsqueeze(0))
+        if dist_table is not None:
+            att = att + dist_table[(qi - kj).clamp(0, dist_table.shape[0] - 1)].permute(2, 0, 1)
         dead = kj > qi
         if window is not None:
             dead = dead | (qi - kj >= window)
@@ -703,16 +710,43 @@ def qk_norm_rope_kv_write(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, 
                           k_cache: torch.Tensor, v_cache: torch.Tensor, slots: torch.Tensor,
                           freqs: Optional[torch.Tensor] = None, mag: float = 1.0, unit_norm: bool = False,
                           angles: Optional[torch.Tensor] = None,
-                          v_angles: Optional[torch.Tensor] = None) -> torch.Tensor:
+                          v_angles: Optional[torch.Tensor] = None, whole_norm: bool = False,
+                          q_temp: Optional[Tuple[float, int]] = None, v_mix=None) -> torch.Tensor:
     """qkv [T, >= H*D + G*D + G*Dv] = [queries | keys | values]. Per-head RMS norm of q and k (weights optional),
     then the rotate-half rotation of both; rotated keys go to the K cache, values as projected to the V cache.
     Returns the queries [T, H * D]. With num_kv_heads == 0 the row holds queries only (a layer that reads another
     layer's keys and values) and no cache is touched. `freqs`, `mag`: see `rotate_half_pairs`. `unit_norm`: q and k
     are divided by their root mean square per head without a weight. `angles` [T, rot_dims] fp32 (cos | sin per pair,
     see `rotary_angles`) replaces the base / frequencies; `v_angles` [T, v_dim] likewise: the values are rotated too,
-    over their whole width, and cached so."""
+    over their whole width, and cached so. `whole_norm`: the RMS norms run over all rows of q (of k) at once, with
+    weights [H * D] ([G * D]). `q_temp` (coef, every): q at position p times 1 + coef ln(floor((p + 1) / every) + 1), last.
+    `v_mix` (first, lam): the cached values are (1 - lam) v + lam first, first [T, G * Dv] (any row stride) the values of
+    another layer, lam a one-element fp32 tensor."""
     t = qkv.shape[0]
     hd, gd = num_heads * dim, num_kv_heads * dim
+    if whole_norm or q_temp is not None or v_mix is not None:
+        assert num_kv_heads > 0 and v_angles is None and not (whole_norm and unit_norm)
+        q, k = qkv[:, :hd].float(), qkv[:, hd:hd + gd].float()
+        v = qkv[:, hd + gd:hd + gd + num_kv_heads * v_dim]
+        if q_norm_w is not None or unit_norm:
+            per = (lambda x: x) if whole_norm else (lambda x: x.unflatten(1, (-1, dim)))
+            q = per(q) * torch.rsqrt((per(q) * per(q)).mean(-1, keepdim=True) + eps) * \
+                (1.0 if unit_norm else q_norm_w.float())
+            k = per(k) * torch.rsqrt((per(k) * per(k)).mean(-1, keepdim=True) + eps) * \
+                (1.0 if unit_norm else k_norm_w.float())
+        q, k = q.reshape(t, num_heads, dim), k.reshape(t, num_kv_heads, dim)
+        if angles is not None:
+            q, k = turn_pairs(q, angles), turn_pairs(k, angles)
+        else:
+            q = rotate_half_pairs(q, positions, rot_dims, rot_base, freqs, mag)
+            k = rotate_half_pairs(k, positions, rot_dims, rot_base, freqs, mag)
+        if q_temp is not None:
+            q = q * query_temperature(positions, *q_temp)[:, None, None]
+        if v_mix is not None:
+            v = ((1.0 - v_mix[1]) * v.float() + v_mix[1] * v_mix[0].float()).to(qkv.dtype)
+        _cache_rows_write(k_cache, slots, k.to(qkv.dtype))
+        _cache_rows_write(v_cache, slots, v.reshape(t, num_kv_heads, v_dim))
+        return q.to(qkv.dtype).reshape(t, hd)
     if unit_norm:
         q_norm_w = k_norm_w = torch.ones(dim, device=qkv.device)
     if angles is not None or v_angles is not None:
@@ -741,6 +775,25 @@ def qk_norm_rope_kv_write(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, 
     _cache_rows_write(k_cache, slots, k.to(qkv.dtype))
     _cache_rows_write(v_cache, slots, v)
     return q.to(qkv.dtype).reshape(t, hd)
+
+
+def query_temperature(positions: torch.Tensor, coef: float, every: int) -> torch.Tensor:
+    """fp32 factor per position p: 1 + coef ln(floor((p + 1) / every) + 1)."""
+    step = (positions + 1).div(every, rounding_mode="floor") + 1
+    return 1.0 + coef * torch.log(step.float())
+
+
+def distance_buckets(rows: int, dmax: float) -> List[int]:
+    """Table row per distance 0, 1, ...: the first half of the `rows` has one distance each, the others grow
+    logarithmically up to `dmax` and the last one takes everything beyond. The list ends with the first distance of the
+    last row (every farther one has the same row). Formed in double precision."""
+    half = rows // 2
+    assert rows >= 1 and (half == 0 or dmax > half), (rows, dmax)
+    out = list(range(half))
+    while half and (not out or out[-1] < rows - 1):
+        n = len(out)
+        out.append(min(rows - 1, half + math.floor(math.log(n / half) / math.log(dmax / half) * (rows - half))))
+    return out or [0]
 
 
 def linear_state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: Optional[torch.Tensor],
@@ -865,18 +918,29 @@ def ssd_scan(x: torch.Tensor, b: torch.Tensor, c: torch.Tensor, dt: torch.Tensor
     return out
 
 
+def gate_rows(o: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
+    """In place: o [T, n] times sigmoid(gate [T, n]) (any row stride)."""
+    return o.copy_((o.float() * torch.sigmoid(gate.float())).to(o.dtype))
+
+
 def gelu_gate_embed(g: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, col0: int) -> torch.Tensor:
     """gelu_tanh(g) * table[ids, col0 : col0 + dim] for g [T, dim]."""
     e = table[ids.long(), col0:col0 + g.shape[1]]
     return (F.gelu(g.float(), approximate="tanh") * e.float()).to(g.dtype)
 
 
-def silu_mul(gu: torch.Tensor, block: int = 0) -> torch.Tensor:
-    """gu [T, 2F] = [gate | up] -> silu(gate) * up. `block` > 0: blocks of gate and up columns alternate."""
+def _gate_act(g: torch.Tensor, act: str) -> torch.Tensor:
+    assert act in ("silu", "gelu"), act
+    return F.silu(g) if act == "silu" else F.gelu(g, approximate="tanh")
+
+
+def silu_mul(gu: torch.Tensor, block: int = 0, act: str = "silu") -> torch.Tensor:
+    """gu [T, 2F] = [gate | up] -> silu(gate) * up. `block` > 0: blocks of gate and up columns alternate. `act`
+    "gelu": the tanh form of gelu instead of silu."""
     f = gu.shape[1] // 2
     if block:
         gu = gu.reshape(gu.shape[0], f // block, 2, block).transpose(1, 2).reshape(gu.shape[0], 2 * f)
-    return (F.silu(gu[:, :f].float()) * gu[:, f:].float()).to(gu.dtype)
+    return (_gate_act(gu[:, :f].float(), act) * gu[:, f:].float()).to(gu.dtype)
 
 
 def router_topk(h: torch.Tensor, w: torch.Tensor, top_k: int):
@@ -969,10 +1033,14 @@ def banded_rotary_frequencies(dims: int, base: float, scaling: Optional[dict] = 
                               dtype=torch.float64) -> torch.Tensor:
     """Frequency per pair with Llama 3.1 style `scaling` {factor, low, high, original}: by wavelength 2 pi / f, short
     waves (< original / high) keep f, long ones (> original / low) take f / factor, those between are blended by
-    s = (original / wavelength - low) / (high - low): (1 - s) f / factor + s f."""
+    s = (original / wavelength - low) / (high - low): (1 - s) f / factor + s f. `scaling` with a factor alone is linear:
+    every frequency is divided by it."""
     i = torch.arange(dims // 2, dtype=torch.float64)
     f = torch.exp(-(2.0 * i / max(dims, 1)) * math.log(base))
-    if scaling:
+    if scaling and "low" not in scaling:
+        assert set(scaling) <= {"factor", "type", "kind"}, scaling
+        f = f / float(scaling["factor"])
+    elif scaling:
         factor, low, high, orig = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
         wave = 2.0 * math.pi / f
         s = (orig / wave - low) / (high - low) if high != low else torch.zeros_like(f)
@@ -1011,28 +1079,36 @@ def linear_batched(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch
 
 def latent_norm_rope_write(q: torch.Tensor, dkv: torch.Tensor, rank: int, rot: int, norm_w: torch.Tensor, eps: float,
                            positions: torch.Tensor, freqs: torch.Tensor, mag: float, q_full: torch.Tensor,
-                           cache: Optional[torch.Tensor], slots: Optional[torch.Tensor]):
+                           cache: Optional[torch.Tensor], slots: Optional[torch.Tensor],
+                           angles: Optional[torch.Tensor] = None):
     """Latent attention, between the projections and the attention: q [T, H, dim + rot] (view) — its last `rot`
     entries per head are rotated into q_full[:, :, rank:] (q_full [T, H, rank + rot]; the first `rank` columns are
     the caller's: the absorbed queries). dkv [T, rank + rot]: the first `rank` columns are RMS-normed with norm_w
     (the latent), the last `rot` rotated (the key part all heads share); the row [latent | rotated key] goes to
     the paged latent cache [pages, 1, (rank + rot) / slab, page, slab] at `slots`. Norm, angles and rotation in
-    fp32."""
+    fp32. Without `angles` the pairs are neighbours (2i, 2i + 1) and the angle is formed here; with `angles` [T, rot] (cos |
+    sin per pair, `rotary_angles`) the pairs are (i, i + rot / 2)."""
     t, h = q.shape[0], q.shape[1]
     dim = q.shape[2] - rot
-    q_full[:, :, rank:] = rotate_adjacent_pairs(q[:, :, dim:].float(), positions, freqs, mag).to(q_full.dtype)
+
+    def turn(x):
+        return turn_pairs(x, angles) if angles is not None else rotate_adjacent_pairs(x, positions, freqs, mag)
+
+    q_full[:, :, rank:] = turn(q[:, :, dim:].float()).to(q_full.dtype)
     c = dkv[:, :rank].float()
     c = c * torch.rsqrt((c * c).mean(-1, keepdim=True) + eps) * norm_w.float()
-    kr = rotate_adjacent_pairs(dkv[:, rank:rank + rot].float(), positions, freqs, mag)
+    kr = turn(dkv[:, None, rank:rank + rot].float())[:, 0]
     if cache is not None:
         _cache_rows_write(cache, slots, torch.cat([c, kr], -1).to(cache.dtype).reshape(t, 1, rank + rot))
 
 
 def latent_attention(q_full: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, seq_lens: torch.Tensor,
-                     query_start_loc: torch.Tensor, scale: float, rank: int) -> torch.Tensor:
+                     query_start_loc: torch.Tensor, scale: float, rank: int, window: Optional[int] = None,
+                     sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal multi-query attention over the paged latent cache: every head's query q_full [T, H, rank + rot]
     meets the one shared key row [latent | rotated key]; the values are the row's first `rank` columns.
-    -> out [T, H, rank] in q_full's dtype. Scores and softmax in fp32."""
+    -> out [T, H, rank] in q_full's dtype. Scores and softmax in fp32. `window`: position i sees j with
+    0 <= i - j < window; `sink` [H] fp32: one more logit per head in the denominator that carries no value."""
     t, h, d = q_full.shape
     out = torch.zeros(t, h, rank, dtype=q_full.dtype, device=q_full.device)
     qsl, sl = query_start_loc.tolist(), seq_lens.tolist()
@@ -1045,8 +1121,14 @@ def latent_attention(q_full: torch.Tensor, cache: torch.Tensor, block_table: tor
         att = torch.einsum("qhd,kd->hqk", q_full[q0:q1].float(), lat) * scale
         qi = torch.arange(ql, device=q_full.device).view(ql, 1) + (sl[s] - ql)
         kj = torch.arange(sl[s], device=q_full.device).view(1, sl[s])
-        att = att.masked_fill((kj > qi).unsqueeze(0), float("-inf"))
-        out[q0:q1] = torch.einsum("hqk,kd->qhd", torch.softmax(att, -1), lat[:, :rank]).to(q_full.dtype)
+        dead = kj > qi
+        if window is not None:
+            dead = dead | (qi - kj >= window)
+        att = att.masked_fill(dead.unsqueeze(0), float("-inf"))
+        if sink is not None:
+            att = torch.cat([att, sink.float().view(h, 1, 1).expand(h, ql, 1)], dim=-1)
+        p = torch.softmax(att, -1)[..., :sl[s]]
+        out[q0:q1] = torch.einsum("hqk,kd->qhd", p, lat[:, :rank]).to(q_full.dtype)
     return out
 
 

@@ -57,13 +57,14 @@ def _smallm_workspace(device):
     return ws
 
 
-def _linear_smallm(x, w, bias, out, silu: bool):
+def _linear_smallm(x, w, bias, out, silu: int):
+    """`silu`: 0 plain, 1 SiLU-gate, 2 tanh-gelu-gate (gate / up rows interleaved per 128)."""
     m, k = x.shape
     n = w.shape[0]
     ws, cnt, _ = _smallm_workspace(x.device)
     L = _lib.load()
     rc = L.gllm_gemm_smallm(_p(x), x.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), m, n, k, _p(bias),
-                            1 if silu else 0, _FORCE_SPLIT, _p(ws), ws.numel(), _p(cnt), stream_ptr())
+                            int(silu), _FORCE_SPLIT, _p(ws), ws.numel(), _p(cnt), stream_ptr())
     check(rc, "gemm_smallm")
     _count()
     return out
@@ -85,7 +86,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     if m == 0:
         return out
     if comm is None and epi == 0 and _FORCE_BN == 0 and (m <= _SMALLM_MAX or (m <= 64 and k >= 8192)):
-        return _linear_smallm(x, w, bias, out, False)
+        return _linear_smallm(x, w, bias, out, 0)
     L = _lib.load()
     ws, _, tcnt = _smallm_workspace(x.device)
     rc = L.gllm_gemm_bf16(_p(x), x.stride(0), _p(w), w.stride(0), _p(out), out.stride(0), m, n, k, _p(bias),
@@ -97,8 +98,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
 
 
 def linear_silu_mul(x: torch.Tensor, w_interleaved: torch.Tensor, out: Optional[torch.Tensor] = None,
-                    comm: Optional[GemmComm] = None):
-    """Fused gate/up projection + SiLU-gate epilogue; weight rows interleaved per 128
+                    comm: Optional[GemmComm] = None, act: str = "silu"):
+    """Fused gate/up projection + gated epilogue (`act` "silu" | "gelu", the tanh form); weight rows interleaved per 128
     (see ops.ref.interleave_gate_up): BN=256 tiles == [128 gate | 128 up] (the 128-wide tile is
     SMEM-bandwidth bound: 934 us vs 534 us for the Qwen3-8B gate/up GEMM at M=4096)."""
     assert x.dtype == _BF16 and w_interleaved.dtype == _BF16
@@ -109,9 +110,18 @@ def linear_silu_mul(x: torch.Tensor, w_interleaved: torch.Tensor, out: Optional[
     if m == 0:
         return out
     if m <= _SMALLM_MAX and _FORCE_BN == 0 and comm is None:
-        return _linear_smallm(x, w_interleaved, None, out, True)
+        return _linear_smallm(x, w_interleaved, None, out, 1 if act == "silu" else 2)
     L = _lib.load()
     ws, _, tcnt = _smallm_workspace(x.device)
+    if act == "gelu":
+        assert comm is None
+        rc = L.gllm_gemm_bf16_gelu(_p(x), x.stride(0), _p(w_interleaved), w_interleaved.stride(0), _p(out),
+                                   out.stride(0), m, n, k, _p(ws), ws.numel() * 4, _p(tcnt), _SPLITK_MAX_TILES,
+                                   stream_ptr())
+        check(rc, "gemm_bf16_gelu")
+        _count()
+        return out
+    assert act == "silu", act
     rc = L.gllm_gemm_bf16(_p(x), x.stride(0), _p(w_interleaved), w_interleaved.stride(0), _p(out),
                           out.stride(0), m, n, k, None, 1, 256,
                           ctypes.byref(comm) if comm is not None else None, _p(ws), ws.numel() * 4, _p(tcnt),
@@ -496,16 +506,21 @@ def mla_rope_cache(q_pe: torch.Tensor, q_full: torch.Tensor, k_pe: torch.Tensor,
 
 def mla_attention(q_full: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor,
                   tok_seq: Optional[torch.Tensor], positions: torch.Tensor, scale: float,
-                  splits: Optional[int] = None) -> torch.Tensor:
-    """q_full [T,H,576] bf16 -> out_lat [T,H,512]; every token attends to keys [0, position]."""
+                  splits: Optional[int] = None, window: Optional[int] = None,
+                  sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """q_full [T,H,576] bf16 -> out_lat [T,H,512]; every token attends to keys [0, position], or the last `window` of
+    them; `sink` [H] fp32: one more logit per head in the softmax denominator, without a value."""
     t, h, d = q_full.shape
     assert d == 576 and q_full.is_contiguous() and q_full.dtype == _BF16
     pages, hkv, nslab, page_size, w = cache.shape
     assert hkv == 1 and nslab == 9 and w == 64
     if positions.dim() == 2:
         positions = positions[0]
+    assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous())
     if splits is None:
         splits = mla_splits(t, h)
+        if window:
+            splits = max(1, min(splits, (window + 63) // 64))
     out = torch.empty(t, h, 512, dtype=_BF16, device=q_full.device)
     part_o = part_lse = None
     if splits > 1:
@@ -517,6 +532,6 @@ def mla_attention(q_full: torch.Tensor, cache: torch.Tensor, block_table: torch.
     L = _lib.load()
     check(L.gllm_mla_attention(_p(q_full), _p(out), _p(cache), pages, _p(block_table), _p(tok_seq), _p(positions),
                                _p(part_o), _p(part_lse), t, block_table.shape[1], h, page_size, splits, float(scale),
-                               stream_ptr()), "mla_attention")
+                               int(window or 0), _p(sink), stream_ptr()), "mla_attention")
     _count(2 if splits > 1 else 1)
     return out

@@ -33,8 +33,9 @@ def _L():
             "gllm_lat_rms_rows": [P, G, P, P, I, I, F, I, P],
             "gllm_lat_gemm_batched": [P, G, G, P, G, G, P, G, G, I, I, I, I, I, I, P],
             "gllm_lat_rglru_scan": [P, P, P, P, P, G, P, P, P, P, P, I, I, I, P, I, I, P, I, P],
-            "gllm_lat_norm_rope_write": [P, G, G, I, I, P, G, I, I, P, F, P, P, F, P, P, P, I, I, I, I, P],
-            "gllm_lat_attention": [P, P, P, I, P, P, I, I, F, I, I, I, P, I, I, I, P],
+            "gllm_lat_norm_rope_write": [P, G, G, I, I, P, G, I, I, P, F, P, P, F, P, P, P, I, I, I, I, P, P],
+            "gllm_lat_attention": [P, P, P, I, P, P, I, I, F, I, I, I, P, I, I, I, I, P, P],
+            "gllm_lat_gate_rows": [P, G, P, G, I, I, I, P],
             "gllm_lat_grouped_router_select": [P, P, I, I, I, I, I, F, P, P, I, I, I, P],
             "gllm_lat_glu_clamp": [P, G, I, I, P, F, F, I, P],
             "gllm_lat_identity_experts_add": [P, G, P, P, I, I, I, I, P, I, P],
@@ -147,22 +148,37 @@ def rglru_scan(u, gates, gate_bias, c_decay, y_pre, y_bias, state, rec_slots, se
     return out
 
 
-def latent_norm_rope_write(q, dkv, rank, rot, norm_w, eps, positions, freqs, mag, q_full, cache, slots):
+def gate_rows(o, gate):
+    t, n = o.shape
+    assert o.stride(1) == 1 and gate.stride(1) == 1 and gate.shape == (t, n) and gate.dtype == o.dtype
+    check(_L().gllm_lat_gate_rows(_p(o), o.stride(0), _p(gate), gate.stride(0), t, n, _f32(o), stream_ptr()),
+          "lat_gate_rows")
+    sm100._count()
+    return o
+
+
+def latent_norm_rope_write(q, dkv, rank, rot, norm_w, eps, positions, freqs, mag, q_full, cache, slots, angles=None):
     t, h = q.shape[0], q.shape[1]
     dim = q.shape[2] - rot
     assert q.stride(2) == 1 and dkv.stride(1) == 1 and q_full.is_contiguous() and q_full.shape == (t, h, rank + rot)
-    assert freqs.dtype == torch.float32 and freqs.shape[0] == rot // 2 and positions.dim() == 1
+    assert freqs.shape[0] == rot // 2 and positions.dim() == 1
+    if angles is None:
+        assert freqs.dtype == torch.float32
+    else:
+        assert angles.dtype == torch.float32 and angles.is_contiguous() and angles.shape == (t, rot)
+        freqs = None
     assert cache is None or (cache.dtype == q.dtype and cache.shape[1] == 1)
     ps, slab = (cache.shape[3], cache.shape[4]) if cache is not None else (1, rank + rot)
     check(_L().gllm_lat_norm_rope_write(_p(q), q.stride(0), q.stride(1), h, dim, _p(dkv), dkv.stride(0), rank, rot,
                                         _p(norm_w), float(eps), _p(positions), _p(freqs), float(mag), _p(q_full),
                                         _p(cache), _p(slots if cache is not None else None), ps, slab, t, _f32(q),
-                                        stream_ptr()), "lat_norm_rope_write")
+                                        _p(angles), stream_ptr()), "lat_norm_rope_write")
     sm100._count()
 
 
-def latent_attention(q_full, cache, inp, scale, rank, plain: bool = False):
-    """Causal multi-query attention over the latent cache. bf16 with a 512-wide latent and a 64-wide rotated part
+def latent_attention(q_full, cache, inp, scale, rank, plain: bool = False, window: Optional[int] = None,
+                     sink: Optional[torch.Tensor] = None):
+    """Causal (or sliding-window) multi-query attention over the latent cache. bf16 with a 512-wide latent and a 64-wide rotated part
     (pages of 8 to 64 tokens) runs on the tensor-core latent kernel (csrc/attn/mla_attention.cu, split over the keys
     for small batches);
     every other shape and fp32 on the plain kernel."""
@@ -170,12 +186,14 @@ def latent_attention(q_full, cache, inp, scale, rank, plain: bool = False):
     assert q_full.is_contiguous() and cache.dtype == q_full.dtype
     ps, slab = cache.shape[3], cache.shape[4]
     if not plain and q_full.dtype == _BF16 and rank == 512 and dl == 576 and slab == 64 and ps >= 8 and 64 % ps == 0:
-        return sm100.mla_attention(q_full, cache, inp.block_table, inp.tok_seq, inp.positions, scale)
+        return sm100.mla_attention(q_full, cache, inp.block_table, inp.tok_seq, inp.positions, scale, window=window,
+                                   sink=sink)
+    assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.shape[0] == h)
     out = torch.empty(t, h, rank, dtype=q_full.dtype, device=q_full.device)
     bt = inp.block_table
     check(_L().gllm_lat_attention(_p(q_full), _p(cache), _p(bt), bt.stride(0), _p(inp.query_start_loc),
                                   _p(inp.positions), t, inp.seq_lens.shape[0], float(scale), h, dl, rank, _p(out), ps,
-                                  slab, _f32(q_full), stream_ptr()), "lat_attention")
+                                  slab, _f32(q_full), int(window or 0), _p(sink), stream_ptr()), "lat_attention")
     sm100._count()
     return out
 

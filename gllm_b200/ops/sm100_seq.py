@@ -26,19 +26,19 @@ def _L():
         P, I, G, F = c_void_p, c_int, c_long, c_float
         sigs = {
             "gllm_seq_embed_scale": [P, P, P, I, I, I, F, I, P],
-            "gllm_seq_resid_norm": [P, P, G, P, P, P, P, P, I, I, F, I, I, F, F, F, P],
+            "gllm_seq_resid_norm": [P, P, G, P, P, P, P, P, I, I, F, I, I, F, F, F, I, P],
             "gllm_seq_qk_norm_kv_write": [P, G, I, I, I, I, P, P, F, P, P, P, P, I, I, I, P],
             "gllm_seq_window_attention": [P, P, P, P, I, P, P, I, I, F, I, I, I, I, I, I, P, P, G, F, I, I, I, I, F, P, P, P, G,
-                                          P, P],
+                                          P, P, I, P],
             "gllm_seq_postnorm": [P, P, G, P, P, I, I, F, F, I, P],
             "gllm_seq_qk_norm_rope_kv_write": [P, G, I, I, I, I, I, P, P, F, P, I, ctypes.c_double, P, P, P, P, I, I, I,
-                                               I, P, F, I, P, P, P],
+                                               I, P, F, I, P, P, I, F, I, P, G, P, P],
             "gllm_seq_linear_state": [P, G, P, G, P, G, P, G, P, G, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, P,
                                       I, I, P, G, I, P, P],
             "gllm_seq_key_decay": [P, G, P, F, P, I, I, I, P],
             "gllm_seq_gemm_mma_f32out": [P, G, G, P, G, G, P, G, G, I, I, I, I, P],
             "gllm_seq_gated_group_norm": [P, I, P, G, P, I, I, F, I, F, P, G, I, I, P],
-            "gllm_seq_silu_mul": [P, G, I, I, P, G, I, I, P],
+            "gllm_seq_silu_mul": [P, G, I, I, P, G, I, I, I, P],
             "gllm_seq_router_select": [P, I, I, I, P, P, P],
             "gllm_seq_router_logits": [P, G, P, I, I, I, P, I, P],
             "gllm_seq_router_logits_mma": [P, G, P, I, I, I, P, P],
@@ -52,10 +52,11 @@ def _L():
             "gllm_attn_decode_win": [P, G, P, P, P, G, P, P, I, I, I, I, I, I, I, F, I, P, P],
             "gllm_attn_prefill_win": [P, G, P, P, P, G, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P],
             "gllm_attn_prefill_tc_cap": [P, G, P, P, P, G, P, P, P, I, I, I, I, I, I, I, I, F, I, P, F, I, G, P, P, P, G, P,
-                                         P],
-            "gllm_attn_decode_mask": [P, G, P, G, P, P, G, P, P, I, I, I, I, I, I, I, F, I, I, P, F, F, P, P, P, G, P, P],
+                                         P, I, P],
+            "gllm_attn_decode_mask": [P, G, P, G, P, P, G, P, P, I, I, I, I, I, I, I, F, I, I, P, F, F, P, P, P, G, P, P,
+                                      I, P],
             "gllm_attn_prefill_mask": [P, G, P, G, P, P, G, P, P, P, I, I, I, I, I, I, I, I, F, I, I, P, F, F, P, P, P, G, P,
-                                       P],
+                                       P, I, P],
         }
         for name, args in sigs.items():
             fn = getattr(L, name)
@@ -105,7 +106,7 @@ def embedding_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float) -> to
 
 
 def resid_norm(x, y, w_post, add, w_pre, eps, out_dtype, emit_plain=False, post_scale=None, w_offset=0.0,
-               out_mul=1.0, y_mul=1.0):
+               out_mul=1.0, y_mul=1.0, center=False):
     assert x.dtype == torch.float32 and x.is_contiguous()
     t, width = x.shape
     plain = bool(emit_plain) and w_pre is None
@@ -126,7 +127,7 @@ def resid_norm(x, y, w_post, add, w_pre, eps, out_dtype, emit_plain=False, post_
         return x if ret_x else None
     check(_L().gllm_seq_resid_norm(_p(x), _p(y), y.stride(0) if y is not None else 0, _p(w_post), _p(post_scale),
                                    _p(add), _p(w_pre), _p(out), t, width, float(eps), int(plain), is32, float(w_offset),
-                                   float(out_mul), float(y_mul), stream_ptr()),
+                                   float(out_mul), float(y_mul), int(center), stream_ptr()),
           "seq_resid_norm")
     sm100._count()
     return x if ret_x else out
@@ -149,14 +150,14 @@ def window_attention(q, k_cache, v_cache, block_table, seq_lens, query_start_loc
                      simt: bool = False, chunk: Optional[int] = None, v_dim: Optional[int] = None,
                      out_scale: float = 1.0, out: Optional[torch.Tensor] = None, softcap: float = 0.0, dist_bias=None,
                      gate: Optional[torch.Tensor] = None, v_turn: Optional[torch.Tensor] = None,
-                     tc: Optional[bool] = None):
+                     tc: Optional[bool] = None, dist_table: Optional[torch.Tensor] = None):
     """Masked paged attention: sliding window (None / 0 = full causal) and / or chunk mask, optional per-head softmax
     sink, values `v_dim` wide, result times `out_scale` into `out` (any row stride). bf16 with v_dim == head_dim
     in 64 / 128 / 256 and pages of 8..64 tokens runs on the tensor-core paged-attention kernels
     (csrc/attn/paged_attention.cu: the first `num_decode_seqs` sequences, one token each, on the decode kernel, the
     rest on the tcgen05 prefill kernel for head sizes 64 / 128 without a chunk mask, else on the mma.sync prefill
     kernel; `tc=False` keeps the latter); everything else (fp32, other head sizes or page sizes) on the plain kernel.
-    `dist_bias`, `gate`, `v_turn`: see `ops.ref.window_attention`."""
+    `dist_bias`, `dist_table`, `gate`, `v_turn`: see `ops.ref.window_attention`."""
     t = q.shape[0]
     v_dim = head_dim if v_dim is None else v_dim
     if out is None:
@@ -178,7 +179,10 @@ def window_attention(q, k_cache, v_cache, block_table, seq_lens, query_start_loc
         tc_ok = tc_ok and ldg % 4 == 0 and gate.data_ptr() % 8 == 0
     vec16 = out.stride(0) % 8 == 0 and out.data_ptr() % 16 == 0 and \
         (gate is None or (ldg % 8 == 0 and gate.data_ptr() % 16 == 0))
-    extras = (_p(r1), _p(r2), _p(gate), ldg, _p(v_turn))
+    assert dist_table is None or (dist_table.dtype == torch.float32 and dist_table.is_contiguous() and
+                                  dist_table.dim() == 2 and dist_table.shape[1] == num_q_heads and r1 is None)
+    extras = (_p(r1), _p(r2), _p(gate), ldg, _p(v_turn), _p(dist_table),
+              dist_table.shape[0] if dist_table is not None else 0)
     if not simt and tc_ok and q.dtype == torch.bfloat16 and head_dim in (64, 128, 256) and slab == 64 and ps >= 8 and \
             64 % ps == 0 and max_q_len is not None:
         L, st = _L(), stream_ptr()
@@ -271,7 +275,7 @@ def postnorm(x, y, alpha, w, eps, out_dtype):
 
 def qk_norm_rope_kv_write(qkv, num_heads, num_kv_heads, dim, v_dim, q_norm_w, k_norm_w, eps, positions, rot_dims,
                           rot_base, k_cache, v_cache, slots, freqs=None, mag=1.0, unit_norm=False, angles=None,
-                          v_angles=None):
+                          v_angles=None, whole_norm=False, q_temp=None, v_mix=None):
     import math
     t = qkv.shape[0]
     assert qkv.stride(1) == 1 and k_cache.dtype == qkv.dtype and positions.dim() == 1
@@ -281,6 +285,11 @@ def qk_norm_rope_kv_write(qkv, num_heads, num_kv_heads, dim, v_dim, q_norm_w, k_
                               angles.shape == (t, rot_dims))
     assert v_angles is None or (v_angles.dtype == torch.float32 and v_angles.is_contiguous() and
                                 v_angles.shape == (t, v_dim))
+    assert not whole_norm or (q_norm_w.shape[0] == num_heads * dim and k_norm_w.shape[0] == num_kv_heads * dim)
+    first, lam = v_mix if v_mix is not None else (None, None)
+    assert first is None or (first.dtype == qkv.dtype and first.stride(1) == 1 and lam.dtype == torch.float32 and
+                             first.shape == (t, num_kv_heads * v_dim))
+    coef, every = q_temp if q_temp is not None else (0.0, 0)
     q = torch.empty(t, num_heads * dim, dtype=qkv.dtype, device=qkv.device)
     ps = k_cache.shape[3]
     check(_L().gllm_seq_qk_norm_rope_kv_write(_p(qkv), qkv.stride(0), t, num_heads, num_kv_heads, dim, v_dim,
@@ -288,7 +297,8 @@ def qk_norm_rope_kv_write(qkv, num_heads, num_kv_heads, dim, v_dim, q_norm_w, k_
                                               math.log2(rot_base) if rot_dims > 0 else 0.0, _p(q), _p(k_cache),
                                               _p(v_cache), _p(slots), ps, k_cache.shape[4], v_cache.shape[4],
                                               _f32(qkv), _p(freqs), float(mag), int(unit_norm), _p(angles),
-                                              _p(v_angles), stream_ptr()),
+                                              _p(v_angles), int(whole_norm), float(coef), int(every), _p(first),
+                                              first.stride(0) if first is not None else 0, _p(lam), stream_ptr()),
           "seq_qk_norm_rope_kv_write")
     sm100._count()
     return q
@@ -341,13 +351,14 @@ def gated_group_norm(o, gate, w, group, eps, act, out_scale=1.0, out=None, out_d
     return out
 
 
-def silu_mul(gu, out=None, block: int = 0):
-    """gu [T, 2F] = [gate | up], or with `block` alternating blocks of gate and up columns."""
+def silu_mul(gu, out=None, block: int = 0, act: str = "silu"):
+    """gu [T, 2F] = [gate | up], or with `block` alternating blocks of gate and up columns; `act` "silu" | "gelu"."""
+    assert act in ("silu", "gelu"), act
     t, f = gu.shape[0], gu.shape[1] // 2
     out = torch.empty(t, f, dtype=gu.dtype, device=gu.device) if out is None else out
     assert gu.stride(1) == 1 and out.stride(1) == 1 and out.shape == (t, f) and out.dtype == gu.dtype
-    check(_L().gllm_seq_silu_mul(_p(gu), gu.stride(0), t, f, _p(out), out.stride(0), _f32(gu), int(block), stream_ptr()),
-          "seq_silu_mul")
+    check(_L().gllm_seq_silu_mul(_p(gu), gu.stride(0), t, f, _p(out), out.stride(0), _f32(gu), int(block),
+                                 int(act == "gelu"), stream_ptr()), "seq_silu_mul")
     sm100._count()
     return out
 
