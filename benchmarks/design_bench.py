@@ -1,7 +1,7 @@
 """Prefill / decode throughput of a layer-list design beside the closest existing decoder at matched width, depth and
 (roughly) parameter count, through the public `LLM.generate` API with random weights, plus the device time of each
 new kernel against its roofline and against the like kernel of the existing path. Invoked as
-`python bench.py --design saritar|femolix|bevovik|notadra|vikupel` (the default benchmark is untouched).
+`python bench.py --design saritar|femolix|bevovik|notadra|vikupel|liverax` (the default benchmark is untouched).
 
   saritar  beside Qwen3 (GQA attention with q/k norm + gated MLP)
   femolix  beside Qwen3-MoE (rotary GQA attention with q/k norm + routed gated experts)
@@ -11,6 +11,7 @@ new kernel against its roofline and against the like kernel of the existing path
            scores, a unit sink, layers on shared key / value pages, sigmoid group-limited routing, ungated
            squared-ReLU experts and a hashed pair embedding)
   vikupel  beside Saritar and Qwen3 (benchmarks/vikupel_bench.py)
+  liverax  beside Qwen3 and Vikupel (benchmarks/liverax_bench.py)
 
 Prints ONE JSON line: {"design": ..., "sizes": [{"width", ..., "<design>": {...}, "<closest>": {...}}], "kernels": [...]}
 """
@@ -388,6 +389,9 @@ def run(args):
     if getattr(args, "design", "saritar") == "vikupel":
         from benchmarks import vikupel_bench
         return vikupel_bench.run(args, peaks)
+    if getattr(args, "design", "saritar") == "liverax":
+        from benchmarks import liverax_bench
+        return liverax_bench.run(args, peaks)
     vocab = 32000
     kernels = _kernels(peaks)
     sizes = []

@@ -195,9 +195,9 @@ class DictReader:
         return tuple(self.w[name].shape)
 
 
-def drive_mixer(m, h, cuts, page_size=4, device="cpu", dtype=torch.float32, pool=512):
+def drive_mixer(m, h, cuts, page_size=4, device="cpu", dtype=torch.float32, pool=512, prepare=None):
     """One mixer alone through the page / slot managers and the batch builder: `h` [T, width] fed in portions of the
-    sizes `cuts`; -> the mixer's outputs [T, width] (fp32, CPU)."""
+    sizes `cuts`; -> the mixer's outputs [T, width] (fp32, CPU). `prepare(inp, start, count)` runs before each portion."""
     from gllm_b200.input_data import InputData, build_batch
     from gllm_b200.memory_manager import HybridCache, MemoryManager
     from gllm_b200.scheduler import ScheduledSeq
@@ -214,6 +214,8 @@ def drive_mixer(m, h, cuts, page_size=4, device="cpu", dtype=torch.float32, pool
         seq.scheduled_token_num = at + c
         mm.pre_allocate_page([seq])
         inp.load(build_batch([ScheduledSeq(seq, at, c)], page_size, 100))
+        if prepare is not None:
+            prepare(inp, at, c)
         got.append(m(inp, h[at:at + c].to(device=device, dtype=dtype), cache, 0).float().cpu())
         at += c
     assert at == n

@@ -64,11 +64,9 @@ def bucket(n, rows, dmax):
 
 def distance_bias(rel, t, dmax):
     """rel [rows, H] -> [H, T, T] (0 above the diagonal, which no query sees)."""
-    out = torch.zeros(rel.shape[1], t, t, dtype=F64)
-    for i in range(t):
-        for j in range(i + 1):
-            out[:, i, j] = rel[bucket(i - j, rel.shape[0], dmax)]
-    return out
+    per_distance = torch.stack([rel[bucket(n, rel.shape[0], dmax)] for n in range(t)])
+    d = torch.arange(t)[:, None] - torch.arange(t)[None, :]
+    return torch.where(d >= 0, per_distance[d.clamp(min=0)].permute(2, 0, 1), 0.0)
 
 
 def temperature(t, q_temp):
