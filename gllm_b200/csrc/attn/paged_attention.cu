@@ -177,10 +177,21 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_cons
   for (int tile = tile_begin; tile < tile_end; ++tile, ++it) {
     const int s = it % SM::kStages;
     const uint32_t ph = (it / SM::kStages) & 1;
+    const int tok0 = warp * 16;  // this warp's 16 tokens inside the tile
+    float tb[2][4];              // distance table entries of this thread's scores, on their way while the tile arrives
+    if (EX && p.ex.dtab != nullptr) {
+      const bool far_tile = seq_len - (tile + 1) * kTileN >= p.ex.dtab_n - 1;        // every key at the table's end
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          tb[nt][e] = far_tile ? far[e >> 1]
+                               : dist_table_log2(tab[e >> 1], p.ex.dtab_n, p.Hq,
+                                                 seq_len - 1 - (tile * kTileN + tok0 + 2 * t + nt * 8 + (e & 1)));
+    }
     mbar_wait(&full_bar[s], ph);
     const uint32_t sk = smem_u32(smem + s * SM::kStageBytes);
     const uint32_t sv = sk + SM::kTileBytes;
-    const int tok0 = warp * 16;  // this warp's 16 tokens inside the tile
 
     // S = Q K^T  (16 rows x 16 tokens)
     float sc[2][4];
@@ -200,7 +211,6 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_cons
     }
     // mask + online softmax (rows g and g+8)
     const int abs0 = tile * kTileN + tok0 + 2 * t;
-    const bool far_tile = EX && seq_len - (tile + 1) * kTileN >= p.ex.dtab_n - 1;    // every key at the table's end
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt) {
@@ -209,8 +219,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_cons
         const int col = abs0 + nt * 8 + (e & 1);
         float v = p.cap_log2 > 0.f ? p.cap_log2 * tanh_exp(sc[nt][e] * p.scale_over_cap) : sc[nt][e] * p.scale_log2;
         if (EX && p.ex.r1 != nullptr) v -= dist_bias_log2(b1[e >> 1], b2[e >> 1], seq_len - 1 - col);
-        if (EX && p.ex.dtab != nullptr)
-          v += far_tile ? far[e >> 1] : dist_table_log2(tab[e >> 1], p.ex.dtab_n, p.Hq, seq_len - 1 - col);
+        if (EX && p.ex.dtab != nullptr) v += tb[nt][e];
         if (col >= seq_len || col < win_lo) v = -INFINITY;
         sc[nt][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);

@@ -56,13 +56,11 @@ struct TcAttnParams {
 
 // BIAS of the kernel: none, the logarithmic distance bias, the distance table
 enum TcBias : int { kNoBias = 0, kLogBias = 1, kTableBias = 2 };
-static constexpr int kTabHeads = 16;                     // heads per CTA with a distance table (bounds its staging)
+static constexpr int kTabFloats = 8192;                  // staging of a distance table (fits beside four KV stages)
 
 template <int D, int KV, int BIAS>
 struct TcSmem {
-  // distance table: per KV tile the entries of its KV + tokens - 1 distances x GP heads, double buffered
-  static constexpr int kTabFloats = KV * kTabHeads + kTcRows;
-  static constexpr int kTabBytes = BIAS == kTableBias ? 2 * kTabFloats * 4 : 0;
+  static constexpr int kTabBytes = BIAS == kTableBias ? kTabFloats * 4 : 0;
   static constexpr int kQBytes = kTcRows * D * 2;
   static constexpr int kTileBytes = KV * D * 2;            // one K (or V) tile
   static constexpr int kStageBytes = 2 * kTileBytes;
@@ -273,30 +271,28 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
     const int low = p.window > 0 ? lim - p.window + 1 : 0;          // first visible key of this row
     float b1 = 0.f, b2 = 0.f;
     if (BIAS == kLogBias) { b1 = p.ex.r1[head]; b2 = p.ex.r2[head]; }
-    // distance table: entry (tile buffer b, distance offset k, head) at [b][k * GP + head]; the offset of key `key` for
-    // this row is row / GP + KV - 1 - (key - key0), so the lanes of a warp read neighbouring words
+    // distance table: staged once per CTA for every distance that its near tiles meet, [distance - dmin][GP heads], so the
+    // lanes of a warp (tokens x heads) read neighbouring words
     float* stab = reinterpret_cast<float*>(smem + SM::kTabOff);
-    if (BIAS == kTableBias) b1 = dist_table_log2(p.ex.dtab + head, p.ex.dtab_n, p.Hq, p.ex.dtab_n - 1);
+    const int dmin = 2 - KV - toks_per_tile;             // smallest distance of any tile (keys behind the diagonal)
+    if (BIAS == kTableBias) {
+      b1 = dist_table_log2(p.ex.dtab + head, p.ex.dtab_n, p.Hq, p.ex.dtab_n - 1);
+      const int dmax = min(p.ex.dtab_n + KV + toks_per_tile - 3, ctx_len + last_tok);
+      const int total = (dmax - dmin + 1) * p.GP;
+      const int dstep = kTcRows / p.GP;                  // GP divides the row count: a thread keeps its head
+      const float* col = p.ex.dtab + head;
+      int d = dmin + row / p.GP;
+#pragma unroll 4
+      for (int e = row; e < total; e += kTcRows, d += dstep) stab[e] = dist_table_log2(col, p.ex.dtab_n, p.Hq, d);
+      asm volatile("bar.sync 1, 128;" ::: "memory");
+    }
     float m_run = -INFINITY, l_run = 0.f;
     for (int tile = 0; tile < n_tiles; ++tile) {
       const int b = tile & 1;
-      bool far_tile = false;
-      const float* trow = stab;
-      if (BIAS == kTableBias) {
-        // smallest distance of the tile (CTA-uniform); at the table's end every score gets the same entry
-        const int d0 = ctx_len + tok_base - ((tile0 + tile) * KV + KV - 1);
-        far_tile = d0 >= p.ex.dtab_n - 1;
-        if (!far_tile) {
-          float* dst = stab + b * SM::kTabFloats;
-          for (int e = row; e < (KV - 1) * p.GP + kTcRows; e += kTcRows) {
-            const int k = e / p.GP;
-            dst[e] = dist_table_log2(p.ex.dtab + hbase + (e - k * p.GP), p.ex.dtab_n, p.Hq, d0 + k);
-          }
-          // one barrier per tile is enough: buffer b was last read two tiles ago, before the previous barrier
-          asm volatile("bar.sync 1, 128;" ::: "memory");
-          trow = dst + row;
-        }
-      }
+      // smallest distance of the tile (CTA-uniform); at the table's end every score gets the same entry
+      const int d0 = ctx_len + tok_base - ((tile0 + tile) * KV + KV - 1);
+      const bool far_tile = BIAS == kTableBias && d0 >= p.ex.dtab_n - 1;
+      const float* trow = stab + (d0 - dmin) * p.GP + row;      // + (KV - 1 - c) GP: the entry of the tile's key c
       mbar_wait(&s_full[b], (tile >> 1) & 1);
       tc_fence_after();
       const uint32_t t_s = tmem + lane_base + b * KV;
@@ -304,66 +300,52 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
       // CTA-uniform: a diagonal tile, or one that the window of some row starts in
       const bool need_mask = key0 + KV - 1 > ctx_len + tok_base ||
                              (p.window > 0 && key0 < ctx_len + last_tok - p.window + 1);
-      // pass 1: row max
-      float mx = -INFINITY;
-#pragma unroll 1
-      for (int c = 0; c < KV; c += 32) {
-        uint32_t v[32];
-        tmem_ld_32x32(t_s + c, v);
-        tmem_ld_wait();
-        if (BIAS == kLogBias) {
+      uint8_t* pb = sp + b * SM::kPBytes;
+      float alpha, sum;
+      // scores of 32 keys from key c on, in the base-2 domain of the softmax (raw without bias and cap: the scale rides
+      // on the exponent's fma); masked ones are -inf
+      auto scores32 = [&](int c, const uint32_t (&v)[32], float* f) {
+        if (BIAS == kTableBias && !far_tile) {
+          const float* tr = trow + (KV - 1 - c) * p.GP;
 #pragma unroll
-          for (int e = 0; e < 32; ++e) {
-            const int key = key0 + c + e;
-            const float x = fmaf(__uint_as_float(v[e]), p.scale_log2, -dist_bias_log2(b1, b2, lim - key));
-            mx = fmaxf(mx, (key <= lim && key >= low) ? x : -INFINITY);
-          }
-        } else if (BIAS == kTableBias && !far_tile) {
-#pragma unroll
-          for (int e = 0; e < 32; ++e) {
-            const int key = key0 + c + e;
-            const float x = fmaf(__uint_as_float(v[e]), p.scale_log2, trow[(KV - 1 - c - e) * p.GP]);
-            mx = fmaxf(mx, (key <= lim && key >= low) ? x : -INFINITY);
-          }
-        } else if (need_mask) {
-#pragma unroll
-          for (int e = 0; e < 32; ++e)
-            mx = fmaxf(mx, (key0 + c + e <= lim && key0 + c + e >= low) ? __uint_as_float(v[e]) : -INFINITY);
+          for (int e = 0; e < 32; ++e) f[e] = fmaf(__uint_as_float(v[e]), p.scale_log2, tr[-e * p.GP]);
         } else {
 #pragma unroll
-          for (int e = 0; e < 32; ++e) mx = fmaxf(mx, __uint_as_float(v[e]));
+          for (int e = 0; e < 32; ++e) {
+            const float x = __uint_as_float(v[e]);
+            f[e] = BIAS == kTableBias ? fmaf(x, p.scale_log2, b1)
+                   : BIAS == kLogBias ? fmaf(x, p.scale_log2, -dist_bias_log2(b1, b2, lim - (key0 + c + e)))
+                   : CAP ? p.cap_log2 * tanh_exp(x * p.scale_over_cap)
+                         : x;
+          }
         }
-      }
-      // the cap is increasing in the score: the capped maximum is the cap of the raw maximum
-      const float mx_s = BIAS == kLogBias || (BIAS == kTableBias && !far_tile) ? mx
-                         : BIAS == kTableBias ? fmaf(mx, p.scale_log2, b1)
-                         : !CAP ? mx * p.scale_log2
-                              : (mx == -INFINITY ? -INFINITY : p.cap_log2 * tanh_exp(mx * p.scale_over_cap));
-      const float m_new = fmaxf(m_run, mx_s);
-      const float m_use = (m_new == -INFINITY) ? 0.f : m_new;
-      const float alpha = exp2f(m_run - m_use);
-      m_run = m_new;
-      // pass 2: P = exp2(S * scale - m), row sum, bf16 P -> smem (A operand of the PV product)
-      uint8_t* pb = sp + b * SM::kPBytes;
-      float sum = 0.f;
-#pragma unroll 1
-      for (int c = 0; c < KV; c += 32) {
-        uint32_t v[32];
-        tmem_ld_32x32(t_s + c, v);
-        tmem_ld_wait();
-        float f[32];
+        if (need_mask) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e)
+            if (key0 + c + e > lim || key0 + c + e < low) f[e] = -INFINITY;
+        }
+      };
+      constexpr bool kRaw = BIAS == kNoBias && !CAP;
+      auto max32 = [](const float* f) {
+        float m4[4] = {f[0], f[1], f[2], f[3]};
+#pragma unroll
+        for (int e = 4; e < 32; ++e) m4[e & 3] = fmaxf(m4[e & 3], f[e]);
+        return fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
+      };
+      float m_use = 0.f;
+      auto new_max = [&](float mx) {
+        const float m_new = fmaxf(m_run, kRaw ? mx * p.scale_log2 : mx);
+        m_use = (m_new == -INFINITY) ? 0.f : m_new;
+        alpha = exp2f(m_run - m_use);
+        m_run = m_new;
+      };
+      // P = exp2(score - m) of 32 keys -> bf16 in smem (A operand of the PV product); returns their sum
+      auto probs32 = [&](int c, float* f) {
+        float s4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
         for (int e = 0; e < 32; ++e) {
-          float x = BIAS == kLogBias ? exp2f(fmaf(__uint_as_float(v[e]), p.scale_log2,
-                                                  -dist_bias_log2(b1, b2, lim - (key0 + c + e)) - m_use))
-                    : BIAS == kTableBias
-                        ? exp2f(fmaf(__uint_as_float(v[e]), p.scale_log2,
-                                     (far_tile ? b1 : trow[(KV - 1 - c - e) * p.GP]) - m_use))
-                    : CAP ? exp2f(fmaf(p.cap_log2, tanh_exp(__uint_as_float(v[e]) * p.scale_over_cap), -m_use))
-                        : exp2f(fmaf(__uint_as_float(v[e]), p.scale_log2, -m_use));
-          if (need_mask && (key0 + c + e > lim || key0 + c + e < low)) x = 0.f;
-          f[e] = x;
-          sum += x;
+          f[e] = kRaw ? exp2f(fmaf(f[e], p.scale_log2, -m_use)) : exp2f(f[e] - m_use);
+          s4[e & 3] += f[e];
         }
 #pragma unroll
         for (int g = 0; g < 4; ++g) {
@@ -373,6 +355,44 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_
           w.z = pack_bf16(f[g * 8 + 4], f[g * 8 + 5]);
           w.w = pack_bf16(f[g * 8 + 6], f[g * 8 + 7]);
           *reinterpret_cast<uint4*>(pb + a_tile_off(row, (c >> 3) + g)) = w;
+        }
+        return (s4[0] + s4[1]) + (s4[2] + s4[3]);
+      };
+      if constexpr (KV == 64) {
+        // the whole row tile stays in registers: S leaves TMEM once
+        float f[64];
+        {
+          uint32_t v0[32], v1[32];
+          tmem_ld_32x32(t_s, v0);
+          tmem_ld_32x32(t_s + 32, v1);
+          tmem_ld_wait();
+          scores32(0, v0, f);
+          scores32(32, v1, f + 32);
+        }
+        new_max(fmaxf(max32(f), max32(f + 32)));
+        sum = probs32(0, f);
+        sum += probs32(32, f + 32);
+      } else {
+        float mx = -INFINITY;
+#pragma unroll 1
+        for (int c = 0; c < KV; c += 32) {
+          uint32_t v[32];
+          float f[32];
+          tmem_ld_32x32(t_s + c, v);
+          tmem_ld_wait();
+          scores32(c, v, f);
+          mx = fmaxf(mx, max32(f));
+        }
+        new_max(mx);
+        sum = 0.f;
+#pragma unroll 1
+        for (int c = 0; c < KV; c += 32) {
+          uint32_t v[32];
+          float f[32];
+          tmem_ld_32x32(t_s + c, v);
+          tmem_ld_wait();
+          scores32(c, v, f);
+          sum += probs32(c, f);
         }
       }
       l_run = l_run * alpha + sum;
@@ -547,8 +567,10 @@ static int attn_prefill_tc_impl(const void* q, int64_t q_ts, void* out, const vo
   if (num_seqs <= 0 || max_q_len <= 0) return 0;
   if ((D != 64 && D != 128) || (kv_tile != 64 && kv_tile != 128) || page_size < 8 || kv_tile % page_size != 0 ||
       Hq % Hkv != 0 || ((ex.r1 != nullptr || ex.dtab != nullptr) && softcap > 0.f) ||
-      (ex.dtab != nullptr && (ex.r1 != nullptr || kv_tile != 64)))
+      (ex.dtab != nullptr && ex.r1 != nullptr))
     return 2;
+  if (ex.dtab != nullptr) kv_tile = 64;
+  if (kv_tile % page_size != 0) return 2;
   CUtensorMap tk, tv;
   if (get_kv_slab_tmap(k_cache, num_pages, Hkv, D, page_size, &tk)) return 1;
   if (get_kv_slab_tmap(v_cache, num_pages, Hkv, D, page_size, &tv)) return 1;
@@ -559,9 +581,16 @@ static int attn_prefill_tc_impl(const void* q, int64_t q_ts, void* out, const vo
   p.seq_lens = reinterpret_cast<const int32_t*>(seq_lens);
   p.q_start = reinterpret_cast<const int32_t*>(q_start);
   p.max_blocks = max_blocks; p.Hq = Hq; p.Hkv = Hkv; p.G = Hq / Hkv;
-  p.GP = 1;
-  for (int d = (p.G < kTcRows ? p.G : kTcRows); d >= 1; --d)
-    if (p.G % d == 0 && kTcRows % d == 0 && (ex.dtab == nullptr || d <= kTabHeads)) { p.GP = d; break; }
+  p.GP = 0;
+  for (int d = (p.G < kTcRows ? p.G : kTcRows); d >= 1; --d) {
+    // with a distance table: as many heads per CTA as its staged part allows
+    if (p.G % d == 0 && kTcRows % d == 0 &&
+        (ex.dtab == nullptr || (int64_t)(ex.dtab_n + 2 * (kv_tile + kTcRows / d)) * d <= kTabFloats)) {
+      p.GP = d;
+      break;
+    }
+  }
+  if (p.GP == 0) return 2;
   p.page_size = page_size; p.seq_offset = seq_offset;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.cap_log2 = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
