@@ -2,9 +2,7 @@
 // Blackwell-native successor of the mma.sync prefill kernel in paged_attention.cu (same arguments, same
 // paged KV cache; reference call site: gllm/layers/attention.py:49-61, flash_attn_varlen_func on the paged cache).
 //
-// OPT-IN (GLLM_ATTN_TC=1, see ops/sm100.py) until it has been validated on hardware: written and compiled this
-// round on a GPU-less box. tests/test_kernels_gpu.py::test_prefill_attention_tc runs it against the fp32 oracle
-// when the switch is set.
+// The default prefill kernel for head sizes 64 and 128; GLLM_ATTN_TC=0 selects the mma.sync kernel (ops/sm100.py).
 //
 // One CTA = 128 query rows (128/GP tokens x GP heads that share one KV head, GQA-packed like the mma.sync kernel)
 // x the causal prefix of one sequence, walked in tiles of KV keys:

@@ -178,10 +178,9 @@ def latent_norm_rope_write(q, dkv, rank, rot, norm_w, eps, positions, freqs, mag
 
 def latent_attention(q_full, cache, inp, scale, rank, plain: bool = False, window: Optional[int] = None,
                      sink: Optional[torch.Tensor] = None):
-    """Causal (or sliding-window) multi-query attention over the latent cache. bf16 with a 512-wide latent and a 64-wide rotated part
-    (pages of 8 to 64 tokens) runs on the tensor-core latent kernel (csrc/attn/mla_attention.cu, split over the keys
-    for small batches);
-    every other shape and fp32 on the plain kernel."""
+    """Causal or sliding-window multi-query attention over the latent cache, with an optional per-head softmax sink. bf16
+    with a 512-wide latent and a 64-wide rotated part (pages of 8 to 64 tokens) runs on the tensor-core latent kernel
+    (csrc/attn/mla_attention.cu, split over the keys for small batches); every other shape and fp32 on the plain kernel."""
     t, h, dl = q_full.shape
     assert q_full.is_contiguous() and cache.dtype == q_full.dtype
     ps, slab = cache.shape[3], cache.shape[4]
